@@ -4,20 +4,26 @@ Each ``csrc/*.cu`` is compiled by nvcc (cross-compiles without a GPU) into an ob
 source and the objects are linked into one shared library that ``rpeg_b200.ops._lib`` loads with
 ctypes. Objects are rebuilt only when their source or a header is newer.
 
+``ensure(names)`` is the on-demand form used when a model is loaded: the full library if it is there and up to date,
+otherwise a library of just the named sources (the kernels one model family launches), compiled on first use.
+
 Run ``python -m rpeg_b200.build_ext`` (add ``--verbose`` for ptxas register/spill output).
 """
 from __future__ import annotations
 
 import concurrent.futures as cf
+import fcntl
 import os
 import shutil
 import subprocess
 import sys
 from pathlib import Path
+from typing import Optional, Sequence
 
 PKG = Path(__file__).resolve().parent
 CSRC = PKG / "csrc"
 LIB = PKG / "librpeg_kernels.so"
+PART_LIB = PKG / "librpeg_part.so"
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -57,9 +63,12 @@ def _compile(src: Path, verbose: bool) -> tuple[Path, str]:
     return obj, res.stderr
 
 
-def build(verbose: bool = False, force: bool = False) -> Path:
-    headers = sorted(CSRC.glob("*.h")) + sorted(CSRC.glob("*.cuh"))
-    srcs = sources()
+def _headers() -> list[Path]:
+    return sorted(CSRC.glob("*.h")) + sorted(CSRC.glob("*.cuh"))
+
+
+def _build(srcs: list[Path], out: Path, verbose: bool, force: bool) -> Path:
+    headers = _headers()
     todo = [s for s in srcs if force or _stale(s.with_suffix(".o"), s, headers)]
     logs: list[str] = []
     if todo:
@@ -67,14 +76,33 @@ def build(verbose: bool = False, force: bool = False) -> Path:
             for obj, log in ex.map(lambda s: _compile(s, verbose), todo):
                 logs.append(f"== {obj.name}\n{log}")
     objs = [s.with_suffix(".o") for s in srcs]
-    if todo or not LIB.exists() or any(o.stat().st_mtime > LIB.stat().st_mtime for o in objs):
-        cmd = [_nvcc(), "-shared", "-o", str(LIB), *map(str, objs), "-lcudart"]
-        res = subprocess.run(cmd, capture_output=True, text=True)
+    if todo or not out.exists() or any(o.stat().st_mtime > out.stat().st_mtime for o in objs):
+        tmp = out.with_suffix(f".{os.getpid()}.tmp.so")
+        res = subprocess.run([_nvcc(), "-shared", "-o", str(tmp), *map(str, objs), "-lcudart"], capture_output=True, text=True)
         if res.returncode != 0:
             raise RuntimeError(f"link failed:\n{res.stdout}\n{res.stderr}")
+        os.replace(tmp, out)
     if verbose:
         print("\n".join(logs))
-    return LIB
+    return out
+
+
+def build(verbose: bool = False, force: bool = False) -> Path:
+    return _build(sources(), LIB, verbose, force)
+
+
+def _fresh(lib: Path, srcs: Sequence[Path]) -> bool:
+    return lib.exists() and all(p.stat().st_mtime <= lib.stat().st_mtime for p in (*srcs, *_headers()))
+
+
+def ensure(names: Optional[Sequence[str]] = None) -> Path:
+    """A loadable library with the kernels of ``csrc/<names>`` (None: all of them); compiles what is missing."""
+    srcs = sources() if names is None else [CSRC / n for n in names]
+    if _fresh(LIB, srcs):
+        return LIB
+    with open(PKG / ".build.lock.tmp", "w") as lock:          # two first calls must not compile into the same objects
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return _build(srcs, LIB if names is None else PART_LIB, False, False)
 
 
 if __name__ == "__main__":

@@ -379,9 +379,13 @@ __device__ __forceinline__ float hash_uniform(uint64_t seed, uint32_t row, uint3
 // One CTA per row: exact multinomial sample from softmax(logits/temp) by the Gumbel-max trick, in
 // the same pass that builds the log-sum-exp, so the sampled token's log-prob costs nothing extra.
 // greedy != 0 picks the argmax. `forced[row] >= 0` overrides the choice (used to inject EOS in
-// synthetic workloads) while still reporting that token's log-prob.
+// synthetic workloads) while still reporting that token's log-prob. Logits are bf16, or fp32 for models that run in fp32.
+__device__ __forceinline__ float logit_at(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ float logit_at(const float* p) { return *p; }
+
+template <typename T>
 __global__ void __launch_bounds__(LP_THREADS)
-sample_kernel(const __nv_bfloat16* __restrict__ logits, int V, int ld, float inv_temp, int greedy,
+sample_kernel(const T* __restrict__ logits, int V, int ld, float inv_temp, int greedy,
               unsigned long long seed, const unsigned long long* __restrict__ seed_offset,
               const int* __restrict__ forced, int* __restrict__ token_out, float* __restrict__ logp_out) {
   griddep_launch();
@@ -391,7 +395,7 @@ sample_kernel(const __nv_bfloat16* __restrict__ logits, int V, int ld, float inv
   const int row = blockIdx.x;
   // a device-resident offset (e.g. a step counter) keeps replays of a captured graph from reusing noise
   if (seed_offset != nullptr) seed += seed_offset[0] * 0xD1B54A32D192ED03ull;
-  const __nv_bfloat16* lr = logits + static_cast<size_t>(row) * ld;
+  const T* lr = logits + static_cast<size_t>(row) * ld;
   float m = -INFINITY, s = 0.f, best = -INFINITY;
   int best_i = 0;
   auto take = [&](int i, float raw) {
@@ -401,7 +405,7 @@ sample_kernel(const __nv_bfloat16* __restrict__ logits, int V, int ld, float inv
     if (!greedy) key += -__logf(-__logf(hash_uniform(seed, row, i)));
     if (key > best || (key == best && i < best_i)) { best = key; best_i = i; }
   };
-  if (((reinterpret_cast<uintptr_t>(lr) | static_cast<uintptr_t>(ld) * 2) & 15) == 0) {
+  if (sizeof(T) == 2 && ((reinterpret_cast<uintptr_t>(lr) | static_cast<uintptr_t>(ld) * 2) & 15) == 0) {
     // 16-byte loads, two in flight per thread: the row is read at memory speed instead of one 2-byte load per
     // round trip (the noise of an element depends on its index only, so the result does not depend on the order)
     const uint4* lv = reinterpret_cast<const uint4*>(lr);
@@ -428,9 +432,9 @@ sample_kernel(const __nv_bfloat16* __restrict__ logits, int V, int ld, float inv
         }
       }
     }
-    for (int i = (nvec << 3) + threadIdx.x; i < V; i += LP_THREADS) take(i, __bfloat162float(lr[i]));
+    for (int i = (nvec << 3) + threadIdx.x; i < V; i += LP_THREADS) take(i, logit_at(lr + i));
   } else {
-    for (int i = threadIdx.x; i < V; i += LP_THREADS) take(i, __bfloat162float(lr[i]));
+    for (int i = threadIdx.x; i < V; i += LP_THREADS) take(i, logit_at(lr + i));
   }
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
 #pragma unroll
@@ -447,7 +451,7 @@ sample_kernel(const __nv_bfloat16* __restrict__ logits, int V, int ld, float inv
       if (sm_best[w] > best || (sm_best[w] == best && sm_idx[w] < best_i)) { best = sm_best[w]; best_i = sm_idx[w]; }
     if (forced != nullptr && forced[row] >= 0) best_i = forced[row];
     token_out[row] = best_i;
-    logp_out[row] = __bfloat162float(lr[best_i]) * inv_temp - (m + __logf(s));
+    logp_out[row] = logit_at(lr + best_i) * inv_temp - (m + __logf(s));
   }
 }
 
@@ -457,8 +461,9 @@ sample_kernel(const __nv_bfloat16* __restrict__ logits, int V, int ld, float inv
 // and no scratch memory is needed (26 passes over a row that stays in L1/L2). The token is then drawn by
 // Gumbel-max among the survivors. The reported log-prob is taken under the FULL softmax, which is what the
 // training passes recompute. top_k <= 0 and top_p >= 1 switch the respective filter off.
+template <typename T>
 __global__ void __launch_bounds__(LP_THREADS)
-sample_filtered_kernel(const __nv_bfloat16* __restrict__ logits, int V, int ld, float inv_temp, int top_k, float top_p,
+sample_filtered_kernel(const T* __restrict__ logits, int V, int ld, float inv_temp, int top_k, float top_p,
                        unsigned long long seed, const unsigned long long* __restrict__ seed_offset,
                        const int* __restrict__ forced, int* __restrict__ token_out, float* __restrict__ logp_out) {
   __shared__ float sm_m[32], sm_s[32], sm_best[32], sm_cnt[32], sm_mass[32];
@@ -466,10 +471,10 @@ sample_filtered_kernel(const __nv_bfloat16* __restrict__ logits, int V, int ld, 
   __shared__ float sm_bc[2];
   const int row = blockIdx.x;
   if (seed_offset != nullptr) seed += seed_offset[0] * 0xD1B54A32D192ED03ull;
-  const __nv_bfloat16* lr = logits + static_cast<size_t>(row) * ld;
+  const T* lr = logits + static_cast<size_t>(row) * ld;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
   float m = -INFINITY, s = 0.f;
-  for (int i = threadIdx.x; i < V; i += LP_THREADS) online_merge(m, s, __bfloat162float(lr[i]) * inv_temp, 1.f);
+  for (int i = threadIdx.x; i < V; i += LP_THREADS) online_merge(m, s, logit_at(lr + i) * inv_temp, 1.f);
   block_lse(m, s, sm_m, sm_s);                       // m, s now hold the row's max and sum(exp(x - m)) in every thread
   const float lse = m + __logf(s);
   const bool use_k = top_k > 0 && top_k < V, use_p = top_p < 1.f;
@@ -479,7 +484,7 @@ sample_filtered_kernel(const __nv_bfloat16* __restrict__ logits, int V, int ld, 
       const float mid_k = 0.5f * (lo_k + hi_k), mid_p = 0.5f * (lo_p + hi_p);
       float cnt = 0.f, mass = 0.f;
       for (int i = threadIdx.x; i < V; i += LP_THREADS) {
-        const float x = __bfloat162float(lr[i]) * inv_temp;
+        const float x = logit_at(lr + i) * inv_temp;
         cnt += x >= mid_k ? 1.f : 0.f;
         mass += x >= mid_p ? __expf(x - lse) : 0.f;
       }
@@ -504,7 +509,7 @@ sample_filtered_kernel(const __nv_bfloat16* __restrict__ logits, int V, int ld, 
   float best = -INFINITY;
   int best_i = 0;
   for (int i = threadIdx.x; i < V; i += LP_THREADS) {
-    const float x = __bfloat162float(lr[i]) * inv_temp;
+    const float x = logit_at(lr + i) * inv_temp;
     if (x < thr) continue;
     const float key = x - __logf(-__logf(hash_uniform(seed, row, i)));
     if (key > best) { best = key; best_i = i; }
@@ -523,7 +528,7 @@ sample_filtered_kernel(const __nv_bfloat16* __restrict__ logits, int V, int ld, 
       if (sm_best[w] > best || (sm_best[w] == best && sm_idx[w] < best_i)) { best = sm_best[w]; best_i = sm_idx[w]; }
     if (forced != nullptr && forced[row] >= 0) best_i = forced[row];
     token_out[row] = best_i;
-    logp_out[row] = __bfloat162float(lr[best_i]) * inv_temp - lse;
+    logp_out[row] = logit_at(lr + best_i) * inv_temp - lse;
   }
 }
 
@@ -665,22 +670,44 @@ extern "C" int rpeg_group_advantage(const float* rewards, float* out, int G, int
   group_advantage_kernel<<<(G + 63) / 64, 64, 0, STREAM(stream)>>>(rewards, out, G, K);
   return LAUNCH_OK();
 }
+template <typename T>
+static int launch_sample(const void* logits, int B, int V, int ld, float temperature, int greedy, unsigned long long seed,
+                         const unsigned long long* seed_offset, const int* forced, int* token_out, float* logp_out, void* stream) {
+  if (B <= 0) return 0;
+  launch_pdl(sample_kernel<T>, dim3(B), dim3(LP_THREADS), 0, STREAM(stream), static_cast<const T*>(logits), V, ld, 1.f / temperature,
+             greedy, seed, seed_offset, forced, token_out, logp_out);
+  return LAUNCH_OK();
+}
+template <typename T>
+static int launch_sample_filtered(const void* logits, int B, int V, int ld, float temperature, int top_k, float top_p,
+                                  unsigned long long seed, const unsigned long long* seed_offset, const int* forced, int* token_out,
+                                  float* logp_out, void* stream) {
+  if (B <= 0) return 0;
+  if (!(temperature > 0.f) || !(top_p > 0.f)) return -2;
+  sample_filtered_kernel<T><<<B, LP_THREADS, 0, STREAM(stream)>>>(static_cast<const T*>(logits), V, ld, 1.f / temperature, top_k, top_p,
+                                                                 seed, seed_offset, forced, token_out, logp_out);
+  return LAUNCH_OK();
+}
 extern "C" int rpeg_sample(const void* logits, int B, int V, int ld, float temperature, int greedy,
                            unsigned long long seed, const unsigned long long* seed_offset, const int* forced,
                            int* token_out, float* logp_out, void* stream) {
-  if (B <= 0) return 0;
-  launch_pdl(sample_kernel, dim3(B), dim3(LP_THREADS), 0, STREAM(stream), static_cast<const __nv_bfloat16*>(logits), V, ld,
-                                                     1.f / temperature, greedy, seed, seed_offset, forced, token_out, logp_out);
-  return LAUNCH_OK();
+  return launch_sample<__nv_bfloat16>(logits, B, V, ld, temperature, greedy, seed, seed_offset, forced, token_out, logp_out, stream);
+}
+extern "C" int rpeg_sample_f32(const void* logits, int B, int V, int ld, float temperature, int greedy,
+                               unsigned long long seed, const unsigned long long* seed_offset, const int* forced,
+                               int* token_out, float* logp_out, void* stream) {
+  return launch_sample<float>(logits, B, V, ld, temperature, greedy, seed, seed_offset, forced, token_out, logp_out, stream);
 }
 extern "C" int rpeg_sample_filtered(const void* logits, int B, int V, int ld, float temperature, int top_k, float top_p,
                                     unsigned long long seed, const unsigned long long* seed_offset, const int* forced,
                                     int* token_out, float* logp_out, void* stream) {
-  if (B <= 0) return 0;
-  if (!(temperature > 0.f) || !(top_p > 0.f)) return -2;
-  sample_filtered_kernel<<<B, LP_THREADS, 0, STREAM(stream)>>>(static_cast<const __nv_bfloat16*>(logits), V, ld, 1.f / temperature,
-                                                              top_k, top_p, seed, seed_offset, forced, token_out, logp_out);
-  return LAUNCH_OK();
+  return launch_sample_filtered<__nv_bfloat16>(logits, B, V, ld, temperature, top_k, top_p, seed, seed_offset, forced, token_out, logp_out,
+                                               stream);
+}
+extern "C" int rpeg_sample_filtered_f32(const void* logits, int B, int V, int ld, float temperature, int top_k, float top_p,
+                                        unsigned long long seed, const unsigned long long* seed_offset, const int* forced,
+                                        int* token_out, float* logp_out, void* stream) {
+  return launch_sample_filtered<float>(logits, B, V, ld, temperature, top_k, top_p, seed, seed_offset, forced, token_out, logp_out, stream);
 }
 extern "C" int rpeg_head_gemv(const void* h, const void* w, const float* bias, float* out, int T, int d,
                               void* stream) {

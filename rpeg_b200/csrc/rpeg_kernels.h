@@ -78,6 +78,11 @@ int rpeg_sample(const void* logits, int B, int V, int ld, float temperature, int
 int rpeg_sample_filtered(const void* logits, int B, int V, int ld, float temperature, int top_k, float top_p,
                          unsigned long long seed, const unsigned long long* seed_offset, const int* forced, int* token_out,
                          float* logp_out, void* stream);
+int rpeg_sample_f32(const void* logits, int B, int V, int ld, float temperature, int greedy, unsigned long long seed,
+                    const unsigned long long* seed_offset, const int* forced, int* token_out, float* logp_out, void* stream);
+int rpeg_sample_filtered_f32(const void* logits, int B, int V, int ld, float temperature, int top_k, float top_p,
+                             unsigned long long seed, const unsigned long long* seed_offset, const int* forced,
+                             int* token_out, float* logp_out, void* stream);
 int rpeg_head_gemv(const void* h, const void* w, const float* bias, float* out, int T, int d, void* stream);
 int rpeg_head_gemv_bwd(const void* h, const void* w, const float* dout, void* dh, float* dw, float* db, int T,
                        int d, void* stream);
@@ -161,6 +166,40 @@ int rpeg_flash_attn_bwd(const void* qkv, int ld, int q_col0, int k_col0, int v_c
                         const void* dout, const float* lse, const int* cu_seqlens, int B, int max_seqlen, int T,
                         int H, int Hkv, int hd, float scale, float* dvec, float* dq_acc, void* dqkv, int ld_dqkv,
                         int* status, void* stream);
+
+// ---- residual_norm.cu: norms around an fp32 residual stream (`kind`: 0 activation, 1 split-K partials, 2 expert outputs,
+// 3 embedding rows, 4 the stream itself); activations and weights are bf16, or fp32 with f32 = 1
+int rpeg_residual_norm(int kind, const void* src, int splits, long long stride, int ld, const int* idx, const float* wts,
+                       int top, int n_shared, long long shared_row0, const void* w, const void* w2, float* x, void* y,
+                       int rows, int d, int dp, float eps, float w_add, int add, int f32, void* stream);
+
+// ---- window_attn.cu / window_prefill.cu: chunked attention with a sink over the paged cache
+int rpeg_rotary_append(const void* src, int splits, long long stride, int ld, int q_col0, int k_col0, int v_col0, const int* slot,
+                       const int* pos, const float* cos_t, const float* sin_t, const int* page_table, int max_pages, void* q_out,
+                       int ldq, void* kcache, void* vcache, int rows, int H, int Hkv, int dim, int dp, int rot_dims, int do_norm,
+                       float eps, int f32, void* stream);
+long long rpeg_rows_attn_scratch(int rows, int H, int dp, int nsplit);
+int rpeg_rows_attn(const void* q, int ldq, const void* kcache, const void* vcache, const int* page_table, int max_pages,
+                   const int* slot, const int* pos, const int* lens, const float* sink, void* out, int ldo, float* scratch,
+                   int* arrive, int rows, int H, int Hkv, int dp, int window, int nsplit, float scale, int f32, int* status,
+                   void* stream);
+int rpeg_window_prefill(const void* q, int ldq, const void* kcache, const void* vcache, long long num_pages, const int* page_table,
+                        int max_pages, const int* cu, const int* pos, const int* slot, const float* sink, void* out, int ldo, int T,
+                        int B, int max_len, int H, int Hkv, int dp, int window, float scale, int* status, void* stream);
+
+// ---- moe.cu: mixture of experts (routing, dispatch, grouped GEMM over the experts' row segments)
+int rpeg_moe_route(const float* logits, int splits, long long stride, int ld, int rows, int E, int n_groups, int keep, int top,
+                   int renorm, int* ids, float* wts, int* ticket, int* counts, void* stream);
+int rpeg_moe_dispatch(const void* x, int dp, const int* ids, const int* ticket, const int* counts, int rows, int E, int top,
+                      void* xs, int* row_of, int* seg_off, int f32, void* stream);
+int rpeg_moe_gemm(const void* A, long long a_rows_total, const void* X, const void* B, void* C, const int* seg_off, int n_routed,
+                  int n_shared, int seg_rows, long long choices, int N, int K, int lda, int ldx, int ldb, int ldc, int gelu,
+                  int bn_hint, int* status, void* stream);
+
+// ---- gemm_f32.cu: fp32 matrix products on the CUDA cores
+int rpeg_gemm_f32(const float* A, const float* B, float* C, int M, int N, int K, int lda, int ldb, int ldc, void* stream);
+int rpeg_moe_gemm_f32(const float* A, const float* X, const float* B, float* C, const int* seg_off, int n_routed, int n_shared,
+                      int seg_rows, int N, int K, int lda, int ldb, int ldc, int gelu, void* stream);
 
 #ifdef __cplusplus
 }

@@ -13,12 +13,16 @@ Design (B200-first):
     bucket graph takes over. Because KV is paged, compaction moves page-table rows, not KV.
   * Sampling log-probs are recorded as the PPO/GRPO ``old_logps`` (no second forward), as in the
     reference (megatron_worker.py:2493-2505).
+Models name their cache layout (``kv_geometry``: heads and widths per layer) and may offer two things more:
+  * ``cached_prefill``: prompts attend over the paged cache, so they can be fed in portions (``prefill_portion`` bounds
+    the tokens of a row one forward takes; ``engine.session`` feeds arbitrary ones);
+  * ``first_visible_key(pos)``: keys below it are never read again (chunked attention). Pages that lie below it are given
+    back to the pool while the row still runs.
 Semantics kept from the reference's quantile-phase generation (:2370-2628): rows end at EOS or at
 the length cap; outputs are returned per original row index, right padded, with a response mask.
 """
 from __future__ import annotations
 
-import math
 from dataclasses import dataclass, field
 from typing import Dict, List, Optional
 
@@ -54,6 +58,11 @@ class PagePool:
         self.free.extend(pages)
 
 
+def page_elems(geometry) -> int:
+    """Elements of one page (keys and values of every layer) under a ``kv_geometry``."""
+    return sum(h * PAGE * (dk + dv) for h, dk, dv in geometry)
+
+
 @dataclass
 class GenerationResult:
     tokens: torch.Tensor        # [N, max_new] int32, right padded with pad_id
@@ -78,33 +87,42 @@ class Generator:
         """Bytes of KV storage that ``slots`` rows of up to ``max_seq_len`` tokens need (+ scratch page) on one of
         ``tp`` tensor-parallel ranks (each keeps its own KV heads)."""
         pages = slots * ((max_seq_len + PAGE - 1) // PAGE) + 1
-        return 2 * cfg.n_layers * pages * (cfg.n_kv_heads // tp) * PAGE * cfg.head_dim * 2
+        return pages * page_elems(cfg.kv_geometry(tp)) * 2
 
     def __init__(self, model: LlamaModel, *, max_slots: int = 64, max_seq_len: int = 2048, kv_budget_bytes: float = 16e9,
                  eos_id: int = 2, pad_id: int = 0, sync_interval: int = 8, use_graphs: bool = True,
-                 kv_storage: Optional[torch.Tensor] = None, group_attention: bool = False):
+                 kv_storage: Optional[torch.Tensor] = None, group_attention: bool = False, prefill_portion: int = 0):
         """``kv_storage``: optional flat bf16 tensor to carve the KV pages from instead of allocating
-        them; lets the cache share memory with buffers that are dead during generation (gradients)."""
+        them; lets the cache share memory with buffers that are dead during generation (gradients).
+        ``prefill_portion``: at most this many tokens of a prompt per forward (0: whole prompts)."""
         cfg = model.cfg
         self.model, self.cfg, self.dev = model, cfg, model.device
         # a tensor-parallel model (models.tp_decode.TPDecodeModel) keeps only its own heads in the cache
         # with peers in the decode step a lost rank must end the loop at the next host sync, not at the length cap
         self.check_status_every_sync = getattr(model, "tp", 1) > 1
-        self.n_kv = getattr(model, "n_kv_local", cfg.n_kv_heads)
-        self.n_heads = getattr(model, "n_heads_local", cfg.n_heads)
+        self.geometry = cfg.kv_geometry(getattr(model, "tp", 1))
+        self.kv_dtype = getattr(model, "dtype", torch.bfloat16)
+        self.cached_prefill = bool(getattr(model, "cached_prefill", False))
+        self.first_visible_key = getattr(model, "first_visible_key", None)
+        if prefill_portion and not self.cached_prefill:
+            raise ValueError("this model prefills whole prompts only")
+        self.prefill_portion = int(prefill_portion)
+        if hasattr(model, "reserve_positions"):
+            model.reserve_positions(max_seq_len)
         self.eos_id, self.pad_id = eos_id, pad_id
         # rows that alias a prompt's KV pages are attended to as a group: the shared keys are read once per group.
         # ``True`` / ``"cuda"``: the CUDA-core group kernel; ``"tc"``: the tcgen05 one (keys on the M axis).
-        self.group_attention = bool(group_attention) and not cfg.qk_norm
+        self.group_attention = bool(group_attention) and not getattr(cfg, "qk_norm", True)
         self.group_tc = str(group_attention).lower() == "tc"
         self.group_min_batch = self.GROUP_MIN_BATCH
         self.sync_interval = max(1, sync_interval)
         self.use_graphs = use_graphs
         self.max_seq_len = max_seq_len
         self.pages_per_row = (max_seq_len + PAGE - 1) // PAGE
-        page_bytes = 2 * cfg.n_layers * self.n_kv * PAGE * cfg.head_dim * 2
+        page_bytes = page_elems(self.geometry) * self.kv_dtype.itemsize
         if kv_storage is not None:
-            kv_budget_bytes = kv_storage.numel() * 2
+            kv_storage = kv_storage.view(self.kv_dtype)
+            kv_budget_bytes = kv_storage.numel() * kv_storage.element_size()
         num_pages = min(int(kv_budget_bytes // page_bytes), max(1, max_slots) * self.pages_per_row + 1)
         if num_pages - 1 < self.pages_per_row:
             raise ValueError(f"KV budget holds {num_pages - 1} pages but one row of {max_seq_len} tokens needs {self.pages_per_row}")
@@ -112,12 +130,19 @@ class Generator:
         # a row that cannot grow because the pool ran dry is preempted and generated again later.
         self.max_slots = max(b for b in (*self.BUCKETS, 4, 2, 1) if b <= max(1, min(max_slots, num_pages - 1)))
         self.pool = PagePool(num_pages)
-        shape = (num_pages, self.n_kv, PAGE, cfg.head_dim)
-        per = math.prod(shape)
+        total = num_pages * page_elems(self.geometry)
+        # a cache carved from someone else's buffer holds arbitrary bits: a model whose kernels load whole pages needs numbers
+        self.zero_cache = kv_storage is not None and bool(getattr(model, "needs_finite_cache", False))
         if kv_storage is None:
-            kv_storage = torch.zeros(2 * cfg.n_layers * per, dtype=torch.bfloat16, device=self.dev)
-        self.kcache = [kv_storage[(2 * l) * per:(2 * l + 1) * per].view(shape) for l in range(cfg.n_layers)]
-        self.vcache = [kv_storage[(2 * l + 1) * per:(2 * l + 2) * per].view(shape) for l in range(cfg.n_layers)]
+            kv_storage = torch.zeros(total, dtype=self.kv_dtype, device=self.dev)
+        self.kv_storage = kv_storage[:total]
+        self.kcache, self.vcache = [], []
+        off = 0
+        for h, dk, dv in self.geometry:
+            for cache, width in ((self.kcache, dk), (self.vcache, dv)):
+                n = num_pages * h * PAGE * width
+                cache.append(kv_storage[off:off + n].view(num_pages, h, PAGE, width))
+                off += n
         n = self.max_slots
         i32 = dict(dtype=torch.int32, device=self.dev)
         self.group_rows = torch.full((n, self.GROUP_MAX), -1, **i32)
@@ -141,11 +166,11 @@ class Generator:
         self.out_lp: Optional[torch.Tensor] = None
         self._graphs: Dict[tuple, torch.cuda.CUDAGraph] = {}
         self._graph_launches: Dict[tuple, int] = {}
-        self.kv_bytes = 2 * cfg.n_layers * math.prod(shape) * 2
+        self.kv_bytes = total * self.kv_dtype.itemsize
 
     # ------------------------------------------------------------------ decode step (graph body)
     def _nsplit(self, b: int) -> int:
-        ctas = b * self.n_heads
+        ctas = b * getattr(self.model, "n_heads_local", getattr(self.cfg, "n_heads", 1))
         return 1 if ctas >= 296 else min(8, (296 + ctas - 1) // ctas)
 
     def _decode_body(self, b: int, temperature: float, greedy: bool, seed: int, top_k: int = 0, top_p: float = 1.0) -> None:
@@ -153,7 +178,8 @@ class Generator:
         # chaining the step's kernels as programmatic dependents hides launch gaps at small batches (-3.7 % at 8 rows)
         # and costs a little once the kernels are long (+0.8 % at 128 rows and more)
         # (a tensor-parallel step is made of short kernels at every batch size: always chained)
-        K.set_pdl(b <= self.PDL_MAX_BATCH or getattr(m, "tp", 1) > 1)
+        # (so is the decode step of a model that asks for it)
+        K.set_pdl(b <= getattr(m, "pdl_max_batch", self.PDL_MAX_BATCH) or getattr(m, "tp", 1) > 1)
         groups = (self.group_rows[:b], self.group_shared[:b], self.row_key0[:b]) if (self.group_attention and b >= self.group_min_batch) else None
         K.set_group_tc(self.group_tc)
         xf = m.decode_step(self.token[:b], self.pos[:b], self.slot_ids[:b], self.seq_len[:b], self.page_table[:b],
@@ -198,15 +224,20 @@ class Generator:
         _lib.add_launches(self._graph_launches[key])
 
     # ------------------------------------------------------------------ prefill of admitted rows
-    def _prefill(self, prompts: List[torch.Tensor], slots: List[int]) -> torch.Tensor:
-        """Run the prompts through the model, store their K/V through the page-table rows of ``slots`` and return
-        the logits at each prompt's last position ``[len(prompts), V]``."""
+    def prefill_hidden(self, pieces: List[torch.Tensor], slots: List[int], starts: Optional[List[int]] = None):
+        """Run one piece of tokens per slot through the model, each continuing at position ``starts[i]`` (0 without it),
+        and store the K/V through the slots' page-table rows. Returns the hidden rows of all pieces and their offsets."""
         cfg, dev = self.cfg, self.dev
-        lens = [int(p.numel()) for p in prompts]
-        tokens = torch.cat(prompts).to(device=dev, dtype=torch.int32)
-        pos = torch.cat([torch.arange(l, dtype=torch.int32) for l in lens]).to(dev)
+        lens = [int(p.numel()) for p in pieces]
+        starts = [0] * len(lens) if starts is None else starts
+        tokens = torch.cat(pieces).to(device=dev, dtype=torch.int32)
+        pos = torch.cat([torch.arange(s, s + l, dtype=torch.int32) for s, l in zip(starts, lens)]).to(dev)
         seq_id = torch.cat([torch.full((l,), s, dtype=torch.int32) for l, s in zip(lens, slots)]).to(dev)
         cu = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32, device=dev)
+        if self.cached_prefill:
+            return self.model.prefill(tokens, pos, cu, max(lens), seq_id, self.page_table, self.kcache, self.vcache), cu
+        if any(starts):
+            raise ValueError("this model prefills whole prompts only")
 
         k_col0, v_col0, n_kv = self.model.kv_columns()
 
@@ -214,9 +245,29 @@ class Generator:
             K.kv_append(qkv, k_col0, v_col0, seq_id, pos, self.page_table, self.kcache[layer],
                         self.vcache[layer], n_kv, cfg.head_dim)
 
-        xf, _ = self.model.forward(tokens, pos, cu, max(lens), keep=False, kv_sink=sink)
-        last = (cu[1:] - 1).contiguous()
-        return self.model.lm_logits(K.gather_rows(xf, last))
+        return self.model.forward(tokens, pos, cu, max(lens), keep=False, kv_sink=sink)[0], cu
+
+    def _prefill(self, prompts: List[torch.Tensor], slots: List[int]) -> torch.Tensor:
+        """Feed the prompts (in portions, if the generator has a limit) and return the logits at each prompt's last
+        position ``[len(prompts), V]``."""
+        n = len(prompts)
+        portion = self.prefill_portion or max(int(p.numel()) for p in prompts)
+        last: List[Optional[torch.Tensor]] = [None] * n
+        done = [0] * n
+        while True:
+            todo = [i for i in range(n) if last[i] is None]
+            if not todo:
+                break
+            pieces = [prompts[i][done[i]:done[i] + portion] for i in todo]
+            xf, cu = self.prefill_hidden(pieces, [slots[i] for i in todo], [done[i] for i in todo])
+            ends = K.gather_rows(xf, (cu[1:] - 1).contiguous())
+            if len(todo) == n and all(p.numel() == q.numel() for p, q in zip(pieces, prompts)):
+                return self.model.lm_logits(ends)
+            for j, i in enumerate(todo):
+                done[i] += int(pieces[j].numel())
+                if done[i] == int(prompts[i].numel()):
+                    last[i] = ends[j]
+        return self.model.lm_logits(torch.stack(last))
 
     def _start_rows(self, logits: torch.Tensor, lens: List[int], slots: List[int], forced: Optional[List[int]], temperature: float,
                     greedy: bool, seed: int, max_new: int, top_k: int = 0, top_p: float = 1.0) -> None:
@@ -281,17 +332,20 @@ class Generator:
         for t in (self.active, self.seq_len, self.gen_count, self.n_finished, self.page_table, self.forced_len):
             t.zero_()
         self.pool = PagePool(self.pool.num_pages)      # a call that raised half way must not leak pages
+        if self.zero_cache:
+            self.kv_storage.zero_()
         self._group_state = None
         self.group_shared.zero_()
         self.row_key0.zero_()
         slot_row = [-1] * n
         slot_pages: List[List[int]] = [[] for _ in range(n)]   # pages a slot owns (the shared prompt pages are not in here)
+        slot_gone = [0] * n        # pages behind the shared ones that the row has passed for good (chunked attention)
         slot_shared = [0] * n      # leading page-table entries that alias the group's shared prompt pages
         slot_bound = [0] * n       # upper bound on the tokens a slot holds (prompt + decode steps run since admission)
         slot_prompt = [0] * n
         queue = list(range(N))
         retired = 0
-        counters = dict(prefill_calls=0, decode_steps=0, prefill_tokens=0, compactions=0, host_syncs=0, kv_pages_taken=0,
+        counters = dict(kv_pages_passed=0, prefill_calls=0, decode_steps=0, prefill_tokens=0, compactions=0, host_syncs=0, kv_pages_taken=0,
                         kv_pages_returned=0, kv_preemptions=0, live_slots_peak=0, graph_replays=0, shared_prompt_pages=0,
                         prompts_prefilled=0)
         seen_finished = 0
@@ -313,7 +367,7 @@ class Generator:
                 self.pool.give(slot_pages[s])
                 slot_pages[s] = []
                 slot_row[s] = -1
-                slot_shared[s] = 0
+                slot_shared[s] = slot_gone[s] = 0
 
         def retire(slots_done: List[int]) -> None:
             nonlocal retired
@@ -356,7 +410,7 @@ class Generator:
             the rows with the least progress when the pool cannot cover it. Returns the rows still live."""
             live = list(live)
             while True:
-                want = {s: pages_for(slot_bound[s] + horizon) - slot_shared[s] - len(slot_pages[s]) for s in live}
+                want = {s: pages_for(slot_bound[s] + horizon) - slot_shared[s] - slot_gone[s] - len(slot_pages[s]) for s in live}
                 total = sum(v for v in want.values() if v > 0)
                 if total <= self.pool.available() or len(live) <= 1:
                     break
@@ -367,7 +421,7 @@ class Generator:
             for s in live:
                 k = want[s]
                 if k > 0:
-                    have = slot_shared[s] + len(slot_pages[s])
+                    have = slot_shared[s] + slot_gone[s] + len(slot_pages[s])
                     new = self.pool.take(k)
                     counters["kv_pages_taken"] += k
                     slot_pages[s].extend(new)
@@ -378,12 +432,31 @@ class Generator:
                                                      torch.tensor(val, dtype=torch.int32, device=dev))
             return live
 
+        def drop_passed(live: List[int]) -> None:
+            """Give back the pages a live row will never read again; its table entries point at the scratch page."""
+            idx: List[int] = []
+            for s in live:
+                first = slot_shared[s] + slot_gone[s]
+                k = min(self.first_visible_key(slot_bound[s] - 1) // PAGE - first, len(slot_pages[s]))
+                if k > 0:
+                    self.pool.give(slot_pages[s][:k])
+                    del slot_pages[s][:k]
+                    slot_gone[s] += k
+                    counters["kv_pages_returned"] += k
+                    counters["kv_pages_passed"] += k
+                    idx.extend(s * self.pages_per_row + first + j for j in range(k))
+            if idx:
+                self.page_table.view(-1)[torch.tensor(idx, dtype=torch.long, device=dev)] = 0
+
         def copy_page(src: int, dst: List[int]) -> None:
             """Copy one KV page (all layers, K and V) onto the pages ``dst``."""
-            per = self.kcache[0].numel()
-            flat = self.kcache[0].new_empty(0).set_(self.kcache[0].untyped_storage(), self.kcache[0].storage_offset(),
-                                                    (2 * self.cfg.n_layers, self.kcache[0].shape[0], per // self.kcache[0].shape[0]))
             d = torch.tensor(dst, dtype=torch.long, device=dev)
+            if len(set(self.geometry)) > 1 or self.geometry[0][1] != self.geometry[0][2]:
+                for c in (*self.kcache, *self.vcache):
+                    c[d] = c[src].unsqueeze(0)
+                return
+            pages = self.kcache[0].shape[0]              # layers of one shape: a single strided copy
+            flat = self.kv_storage.view(2 * self.cfg.n_layers, pages, -1)
             flat[:, d] = flat[:, src].unsqueeze(1)
 
         while retired < N:
@@ -465,9 +538,11 @@ class Generator:
                 break
             used = max(live) + 1
             if not queue and len(live) <= self._bucket(used) // 2 and self._bucket(len(live)) < self._bucket(used):
-                self._compact(live, slot_row, slot_pages, slot_bound, slot_prompt, slot_shared)
+                self._compact(live, slot_row, slot_pages, slot_bound, slot_prompt, slot_shared, slot_gone)
                 counters["compactions"] += 1
                 live = list(range(len(live)))
+            if self.first_visible_key is not None:
+                drop_passed(live)
             live = grow(live)
             used = max(live) + 1
             counters["live_slots_peak"] = max(counters["live_slots_peak"], len(live))
@@ -533,7 +608,7 @@ class Generator:
         return self.max_slots
 
     def _compact(self, live: List[int], slot_row: List[int], slot_pages: List[List[int]], slot_bound: List[int],
-                 slot_prompt: List[int], slot_shared: List[int]) -> None:
+                 slot_prompt: List[int], slot_shared: List[int], slot_gone: List[int]) -> None:
         """Move live slots to the front (state and page-table rows only; KV pages stay where they are)."""
         k = len(live)
         idx = torch.tensor(live, dtype=torch.long, device=self.dev)
@@ -550,8 +625,10 @@ class Generator:
         bounds = [slot_bound[s] for s in live]
         prompts = [slot_prompt[s] for s in live]
         shared = [slot_shared[s] for s in live]
+        gone = [slot_gone[s] for s in live]
         for s in range(len(slot_row)):
             slot_shared[s] = shared[s] if s < k else 0
+            slot_gone[s] = gone[s] if s < k else 0
             slot_row[s] = rows[s] if s < k else -1
             slot_pages[s] = pages[s] if s < k else []
             slot_bound[s] = bounds[s] if s < k else 0

@@ -1,0 +1,373 @@
+"""Dulisun decoder: chunked attention whose values are the projected keys, a softmax sink, norms on the sublayers' outputs
+around an fp32 residual stream, and grouped-router mixtures of experts. Every layer has its own sizes.
+
+    x  = norm(E[token])
+    x += norm1( W_o attention(x) )             q = W_q x, k = W_k x, v = k; interleaved rotary, then unit RMS per head
+    x += norm2( sum_e s_e expert_e(x) + shared(x) )        (layers without a feed-forward skip this)
+    logits = E norm(x)
+
+What runs where:
+  * the residual stream, norms, rotary angles, scores, softmax and routing are fp32; the matrix products take the bf16
+    copy of the stream that the norm kernels write next to it (``dtype=torch.float32`` runs everything in true fp32);
+  * one kernel per place the stream is touched (``ops.kernels.residual_norm``): it sums the split-K partials of the
+    projection before it, or the weighted expert outputs, normalises, adds to the stream and writes the next operand; the
+    norm before the logits rides on the last of them;
+  * keys (rotated, normalised) and values (the raw projection) live in the generator's paged cache. A whole prompt, a
+    portion of one and a decoded token append to it first and then attend over it, so nothing depends on how a prompt was
+    cut. No key before the current chunk is ever read again (``first_visible_key``): the generator gives those pages back;
+  * a shared feed-forward wider than the routed experts is stored as several always-on experts of their size (its hidden
+    units are independent), so routed and shared experts are one grouped GEMM up and one down.
+
+Matrix rows and columns are padded to multiples of 8 elements with zeros (16-byte rows for TMA), so any size loads.
+This family is served (generation, log-probs); it has no backward pass here.
+"""
+from __future__ import annotations
+
+import math
+from dataclasses import dataclass
+from typing import Dict, List, Optional, Tuple
+
+import torch
+
+from ..ops import kernels as K
+from .llama import FlatLayout
+
+
+def pad8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+@dataclass(frozen=True)
+class AttentionMixer:
+    heads: int
+    kv_heads: int
+    dim: int
+    scale: float
+    window: int = 0                     # keys are visible inside chunks of this many positions; 0: all earlier keys
+    rot_dims: int = 0                   # leading dimensions that are rotated (interleaved pairs)
+    rot_base: float = 10000.0
+
+    @property
+    def dim_p(self) -> int:
+        return pad8(self.dim)
+
+    @property
+    def q_width(self) -> int:
+        return self.heads * self.dim_p
+
+    @property
+    def k_width(self) -> int:
+        return self.kv_heads * self.dim_p
+
+
+@dataclass(frozen=True)
+class ExpertMixture:
+    experts: int
+    top: int
+    ff: int
+    shared_ff: int = 0                  # hidden size of the always-on feed-forward; 0: none
+    groups: int = 1
+    keep: int = 1                       # groups a token may choose from
+
+    @property
+    def ff_p(self) -> int:
+        return pad8(self.ff)
+
+    @property
+    def n_shared(self) -> int:
+        """Always-on experts of size ``ff`` that hold the shared feed-forward."""
+        return -(-self.shared_ff // self.ff)
+
+    @property
+    def segments(self) -> int:
+        return self.experts + self.n_shared
+
+
+@dataclass(frozen=True)
+class DecoderLayer:
+    mixer: AttentionMixer
+    mlp: Optional[ExpertMixture] = None
+
+
+@dataclass(frozen=True)
+class DulisunConfig:
+    width: int
+    vocab: int
+    layers: Tuple[DecoderLayer, ...]
+    norm_eps: float = 1e-6
+    max_pos: int = 4096                 # initial size of the rotary tables (they grow with the generator's row length)
+    family: str = "dulisun"
+
+    @property
+    def n_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def d_model(self) -> int:
+        return self.width
+
+    @property
+    def width_p(self) -> int:
+        return pad8(self.width)
+
+    @property
+    def vocab_p(self) -> int:
+        return pad8(self.vocab)
+
+    def kv_geometry(self, tp: int = 1) -> List[Tuple[int, int, int]]:
+        """(KV heads, key width, value width) of every layer's cache."""
+        if tp != 1:
+            raise ValueError("this family has no tensor-parallel cache layout")
+        return [(l.mixer.kv_heads, l.mixer.dim_p, l.mixer.dim_p) for l in self.layers]
+
+    def n_params(self) -> int:
+        return DulisunLayout(self).total
+
+
+class DulisunLayout(FlatLayout):
+    """Flat offsets of every matrix (padded shapes)."""
+
+    def __init__(self, cfg: DulisunConfig):
+        super().__init__()
+        d = cfg.width_p
+        self.add("embed", cfg.vocab_p, d)
+        self.add("embed_norm", d)
+        for i, layer in enumerate(cfg.layers):
+            m, e = layer.mixer, layer.mlp
+            self.add(f"l{i}.wqk", m.q_width + m.k_width, d)
+            self.add(f"l{i}.wo", d, m.q_width)
+            self.add(f"l{i}.norm1", d)
+            if e is not None:
+                self.add(f"l{i}.router", pad8(e.experts), d)
+                self.add(f"l{i}.w_up", e.segments, e.ff_p, d)
+                self.add(f"l{i}.w_down", e.segments, d, e.ff_p)
+                self.add(f"l{i}.norm2", d)
+        self.add("final_norm", d)
+
+
+class DulisunModel:
+    """Weights and kernels of one model on one GPU, with the interface the generator drives."""
+
+    cached_prefill = True               # prompts may be fed in portions: attention reads the paged cache
+    needs_finite_cache = True           # tensor-core tiles cover whole pages: stale entries must be finite numbers
+    KERNEL_SOURCES = ("gemm.cu", "generate.cu", "loss.cu", "residual_norm.cu", "window_attn.cu", "window_prefill.cu", "moe.cu", "gemm_f32.cu")
+
+    def __init__(self, cfg: DulisunConfig, device, *, dtype: torch.dtype = torch.bfloat16, seed: Optional[int] = 0,
+                 trainable: bool = False):
+        """``seed=None`` leaves the weights zero (a checkpoint is about to be loaded)."""
+        if trainable:
+            raise ValueError("the dulisun family has no backward pass: it is served, not trained")
+        if dtype not in (torch.bfloat16, torch.float32):
+            raise ValueError(f"dtype {dtype} is not supported (bfloat16 or float32)")
+        self.cfg, self.device, self.dtype = cfg, torch.device(device), dtype
+        self.f32 = dtype == torch.float32
+        self.layout = DulisunLayout(cfg)
+        self.w = torch.zeros(self.layout.total, dtype=dtype, device=self.device)
+        self.p: Dict[str, torch.Tensor] = {n: self.layout.view(self.w, n) for n in self.layout.entries}
+        self.sink = [torch.zeros(l.mixer.heads, dtype=torch.float32, device=self.device) for l in cfg.layers]
+        self.max_experts = max([l.mlp.experts for l in cfg.layers if l.mlp is not None], default=1)
+        self._ws: Optional[torch.Tensor] = None
+        self._split: Dict[Tuple[int, int], Tuple[torch.Tensor, torch.Tensor]] = {}
+        self._tables: Dict[Tuple[float, int], Tuple[torch.Tensor, torch.Tensor]] = {}
+        self._outgrown: List[dict] = []      # tables that captured graphs may still read
+        self.positions = 0
+        self.reserve_positions(cfg.max_pos)
+        self._num_sms = torch.cuda.get_device_properties(self.device).multi_processor_count if self.device.type == "cuda" else 148
+        if seed is not None:
+            self.init_weights(seed)
+
+    # ------------------------------------------------------------------ weights
+    def init_weights(self, seed: int = 0) -> None:
+        """Random weights of the true sizes (the padding stays zero), unit-gain matrices and norms near one."""
+        gen = torch.Generator(device=self.device)
+        gen.manual_seed(seed)
+
+        def rnd(*shape: int) -> torch.Tensor:
+            return torch.randn(shape, generator=gen, device=self.device, dtype=torch.float32)
+
+        d = self.cfg.width
+        self.p["embed"][: self.cfg.vocab, :d].copy_(rnd(self.cfg.vocab, d) / math.sqrt(d))
+        for name in self.p:
+            if name.endswith(("norm", "norm1", "norm2")):
+                self.p[name][:d].copy_(0.1 * rnd(d))
+        for i, layer in enumerate(self.cfg.layers):
+            m, e = layer.mixer, layer.mlp
+            self.put_qk(i, rnd(m.heads * m.dim, d) / math.sqrt(d), rnd(m.kv_heads * m.dim, d) / math.sqrt(d))
+            self.put_o(i, rnd(d, m.heads * m.dim) / math.sqrt(m.heads * m.dim))
+            self.sink[i].copy_(rnd(m.heads))
+            if e is not None:
+                self.p[f"l{i}.router"][: e.experts, :d].copy_(rnd(e.experts, d) / math.sqrt(d))
+                for s in range(e.experts):
+                    self.put_expert(i, s, rnd(e.ff, d) / math.sqrt(d), rnd(d, e.ff) / math.sqrt(e.ff))
+                if e.shared_ff:
+                    self.put_shared(i, rnd(e.shared_ff, d) / math.sqrt(d), rnd(d, e.shared_ff) / math.sqrt(e.shared_ff))
+
+    def put_qk(self, i: int, wq: torch.Tensor, wk: torch.Tensor) -> None:
+        """Stack the query and key projections, every head padded to ``dim_p`` rows."""
+        m, d = self.cfg.layers[i].mixer, self.cfg.width
+        dst = self.p[f"l{i}.wqk"].view(m.heads + m.kv_heads, m.dim_p, -1)
+        dst[: m.heads, : m.dim, :d].copy_(wq.view(m.heads, m.dim, d))
+        dst[m.heads:, : m.dim, :d].copy_(wk.view(m.kv_heads, m.dim, d))
+
+    def put_o(self, i: int, wo: torch.Tensor) -> None:
+        m, d = self.cfg.layers[i].mixer, self.cfg.width
+        self.p[f"l{i}.wo"].view(-1, m.heads, m.dim_p)[:d, :, : m.dim].copy_(wo.view(d, m.heads, m.dim))
+
+    def put_expert(self, i: int, s: int, up: torch.Tensor, down: torch.Tensor) -> None:
+        """Segment ``s`` of the layer's mixture: up ``[<= ff, width]``, down ``[width, <= ff]``."""
+        d, f = self.cfg.width, up.shape[0]
+        self.p[f"l{i}.w_up"][s, :f, :d].copy_(up)
+        self.p[f"l{i}.w_down"][s, :d, :f].copy_(down)
+
+    def put_shared(self, i: int, up: torch.Tensor, down: torch.Tensor) -> None:
+        """The shared feed-forward, cut along its hidden size into always-on experts of size ``ff``."""
+        e = self.cfg.layers[i].mlp
+        for s in range(e.n_shared):
+            self.put_expert(i, e.experts + s, up[s * e.ff:(s + 1) * e.ff], down[:, s * e.ff:(s + 1) * e.ff])
+
+    # ------------------------------------------------------------------ what the generator asks
+    def kv_geometry(self) -> List[Tuple[int, int, int]]:
+        return self.cfg.kv_geometry()
+
+    def reserve_positions(self, n: int) -> None:
+        """Make the rotary tables cover positions below ``n`` (a generator reserves its longest row when it is built)."""
+        if n <= self.positions:
+            return
+        self.positions = n
+        self._outgrown.append(self._tables)
+        self._tables = {}
+        for l in self.cfg.layers:
+            key = (l.mixer.rot_base, l.mixer.rot_dims)
+            if l.mixer.rot_dims:
+                self._tables[key] = K.rope_tables(n, l.mixer.rot_dims, l.mixer.rot_base, self.device)
+
+    def first_visible_key(self, pos: int) -> int:
+        """Smallest position any layer still reads once every later token stands at ``pos`` or beyond."""
+        return min((pos // l.mixer.window * l.mixer.window if l.mixer.window else 0) for l in self.cfg.layers)
+
+    # ------------------------------------------------------------------ forward
+    def _workspace(self) -> torch.Tensor:
+        if self._ws is None:
+            self._ws = torch.empty(32 * 1024 * 1024, dtype=torch.float32, device=self.device)
+        return self._ws
+
+    def _lin(self, x: torch.Tensor, w: torch.Tensor, decode: bool, f32_out: bool = False):
+        """A projection: split-K partials for few rows (the consumer sums them), a plain GEMM otherwise."""
+        if self.f32:
+            return K.gemm_f32(x, w)
+        if decode:
+            return K.gemm_partials(x, w, self._workspace())
+        return K.gemm(x, w, out_dtype=torch.float32 if f32_out else torch.bfloat16)
+
+    def _mixture(self, i: int, e: ExpertMixture, h: torch.Tensor, counts: torch.Tensor, decode: bool) -> K.MoEOutput:
+        p = self.p
+        logits = self._lin(h, p[f"l{i}.router"], decode, f32_out=True)
+        ids, wts, ticket = K.moe_route(logits, e.experts, e.top, counts, n_groups=e.groups, keep_groups=e.keep)
+        r = K.moe_dispatch(h, ids, wts, ticket, counts, e.experts)
+        act = K.moe_gemm(r.x_sorted, p[f"l{i}.w_up"], r, e.experts, e.n_shared, shared_x=h if e.n_shared else None, gelu=True)
+        y = K.moe_gemm(act, p[f"l{i}.w_down"], r, e.experts, e.n_shared)
+        return K.MoEOutput(y, r.row_of, r.weights, e.n_shared)
+
+    def _run(self, tokens, pos, slot, page_table, kcache, vcache, attend, decode: bool, trace=None) -> torch.Tensor:
+        """All layers on ``T`` tokens; ``attend(layer, q)`` reads the cache after this call appended to it. Returns the
+        hidden rows the logits are taken from, ``[T, width_p]``."""
+        cfg, p, d, eps = self.cfg, self.p, self.cfg.width, self.cfg.norm_eps
+        T = tokens.numel()
+        x = torch.empty((T, cfg.width_p), dtype=torch.float32, device=self.device)
+        counts = torch.zeros((cfg.n_layers, self.max_experts), dtype=torch.int32, device=self.device)
+
+        def norm(src, name: str, last: bool, **kw):
+            y = K.residual_norm(src, p[name], eps, d, x=x, w2=p["final_norm"] if last else None, want_act=not self.f32, **kw)
+            return x if y is None else y
+
+        h = norm(p["embed"], "embed_norm", False, ids=tokens, add=False)
+        for i, layer in enumerate(cfg.layers):
+            m, e = layer.mixer, layer.mlp
+            last = i + 1 == cfg.n_layers
+            cos_t, sin_t = self._tables.get((m.rot_base, m.rot_dims), (None, None))
+            qk = self._lin(h, p[f"l{i}.wqk"], decode)
+            q = torch.empty((T, m.q_width), dtype=self.dtype, device=self.device)
+            K.rotary_append(qk, q, 0, m.q_width, m.q_width, slot, pos, cos_t, sin_t, page_table, kcache[i], vcache[i], m.heads, m.dim,
+                            m.rot_dims, eps)
+            o = self._lin(attend(i, q), p[f"l{i}.wo"], decode)
+            h = norm(o, f"l{i}.norm1", last and e is None)
+            if e is not None:
+                h = norm(self._mixture(i, e, h, counts[i], decode), f"l{i}.norm2", last)
+            if trace is not None:
+                trace.append(x[:, :d].clone())
+        return h
+
+    def prefill(self, tokens, pos, cu, max_len: int, slot, page_table, kcache, vcache, trace=None) -> torch.Tensor:
+        """Packed portions of prompts: request ``b`` owns tokens ``cu[b] .. cu[b + 1]`` at consecutive positions ``pos`` (whatever
+        came before them is in the cache already), ``slot`` names every token's page-table row. Returns hidden rows ``[T, width_p]``."""
+        def attend(i: int, q: torch.Tensor) -> torch.Tensor:
+            m = self.cfg.layers[i].mixer
+            if not self.f32 and m.dim_p <= K.WINDOW_PREFILL_MAX_DIM and m.scale > 0:
+                return K.window_prefill(q, kcache[i], vcache[i], page_table, cu, pos, slot, max_len, m.heads, window=m.window, scale=m.scale,
+                                        sink=self.sink[i])
+            return K.rows_attn(q, kcache[i], vcache[i], page_table, slot, pos, m.heads, window=m.window, scale=m.scale, sink=self.sink[i])
+
+        return self._run(tokens, pos, slot, page_table, kcache, vcache, attend, False, trace)
+
+    def _nsplit(self, m: AttentionMixer, rows: int, table_pages: int) -> int:
+        """Splits that give every SM about two CTAs, at most one per page a row can see."""
+        pages = min(table_pages, m.window // K.KV_PAGE + 2) if m.window else table_pages
+        ctas = rows * m.kv_heads * -(-(m.heads // m.kv_heads) // 8)
+        return max(1, min(-(-2 * self._num_sms // ctas), pages, 32))
+
+    def _split_buffers(self, rows: int, table_pages: int) -> Tuple[torch.Tensor, torch.Tensor]:
+        """Scratch of the split attention for ``rows`` rows; kept for good, captured graphs point into it."""
+        key = (rows, table_pages)
+        if key not in self._split:
+            mixers = [l.mixer for l in self.cfg.layers]
+            need = max(K.rows_attn_scratch(rows, m.heads, m.dim_p, self._nsplit(m, rows, table_pages)) for m in mixers)
+            self._split[key] = (torch.empty(max(need, 1), dtype=torch.float32, device=self.device),
+                                torch.zeros(rows * max(m.heads for m in mixers), dtype=torch.int32, device=self.device))
+        return self._split[key]
+
+    def decode_step(self, token, pos, slot_ids, seq_len, page_table, kcache, vcache, nsplit: int = 1, groups=None) -> torch.Tensor:
+        """One token per row (``seq_len = pos + 1`` visible keys, 0 for a retired row). Returns hidden rows ``[B, width_p]``."""
+        B, table_pages = token.shape[0], page_table.shape[1]
+        scratch, arrive = self._split_buffers(B, table_pages)
+
+        def attend(i: int, q: torch.Tensor) -> torch.Tensor:
+            m = self.cfg.layers[i].mixer
+            return K.rows_attn(q, kcache[i], vcache[i], page_table, slot_ids, pos, m.heads, window=m.window, scale=m.scale, lens=seq_len,
+                               sink=self.sink[i], nsplit=self._nsplit(m, B, table_pages), scratch=scratch, arrive=arrive)
+
+        return self._run(token, pos, slot_ids, page_table, kcache, vcache, attend, True)
+
+    def forward(self, tokens, pos, cu_seqlens, max_seqlen: int, keep: bool = False, kv_sink=None, h_in=None, trace=None):
+        """Packed whole sequences without a generator's cache: the keys go to scratch pages that every layer reuses.
+        ``trace`` (a list) receives the residual stream after every layer."""
+        if keep or kv_sink is not None or h_in is not None:
+            raise ValueError("the dulisun family runs whole sequences for inference only")
+        lens = [int(v) for v in (cu_seqlens[1:] - cu_seqlens[:-1]).tolist()]
+        self.reserve_positions(max(lens))
+        pages = [-(-l // K.KV_PAGE) for l in lens]
+        table = torch.zeros((len(lens), max(pages)), dtype=torch.int32)
+        first = 1
+        for b, n in enumerate(pages):
+            table[b, :n] = torch.arange(first, first + n, dtype=torch.int32)
+            first += n
+        slot = torch.repeat_interleave(torch.arange(len(lens), dtype=torch.int32), torch.tensor(lens)).to(self.device)
+        geom = self.kv_geometry()
+        store = torch.zeros((2, max(first * h * K.KV_PAGE * max(dk, dv) for h, dk, dv in geom)), dtype=self.dtype, device=self.device)
+        kc = [store[0, : first * h * K.KV_PAGE * dk].view(first, h, K.KV_PAGE, dk) for h, dk, _ in geom]
+        vc = [store[1, : first * h * K.KV_PAGE * dv].view(first, h, K.KV_PAGE, dv) for h, _, dv in geom]
+        return self.prefill(tokens, pos, cu_seqlens, max(lens), slot, table.to(self.device), kc, vc, trace), None
+
+    # ------------------------------------------------------------------ heads
+    def lm_logits(self, xf: torch.Tensor, decode: bool = False) -> torch.Tensor:
+        """Logits ``[rows, vocab]`` against the embedding table (bf16, or fp32 in an fp32 model)."""
+        if self.f32:
+            return K.gemm_f32(xf, self.p["embed"])[:, : self.cfg.vocab]
+        return K.gemm(xf, self.p["embed"], workspace=self._workspace() if decode else None)[:, : self.cfg.vocab]
+
+    def token_logprobs(self, xf_rows: torch.Tensor, targets: torch.Tensor, chunk: int = 8192, temperature: float = 1.0) -> torch.Tensor:
+        """``log p(target)`` of the given hidden rows, at most ``chunk`` rows of logits at a time."""
+        out = torch.empty(xf_rows.shape[0], dtype=torch.float32, device=self.device)
+        for s in range(0, xf_rows.shape[0], chunk):
+            t = targets[s:s + chunk].contiguous()
+            _, out[s:s + chunk] = K.sample(self.lm_logits(xf_rows[s:s + chunk]), temperature, True, 0, forced=t)
+        return out

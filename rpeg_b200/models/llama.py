@@ -57,6 +57,10 @@ class LlamaConfig:
     def qkv_width(self) -> int:
         return self.q_width + 2 * self.kv_width
 
+    def kv_geometry(self, tp: int = 1) -> List[Tuple[int, int, int]]:
+        """(KV heads, key width, value width) of every layer's cache on one of ``tp`` tensor-parallel ranks."""
+        return [(self.n_kv_heads // tp, self.head_dim, self.head_dim)] * self.n_layers
+
     def n_params(self) -> int:
         return ParamLayout(self).total
 
@@ -98,26 +102,35 @@ def stage_layers(n_layers: int, stage: Optional[Tuple[int, int]]) -> Tuple[int, 
     return lo, lo + per + (1 if idx < extra else 0)
 
 
-class ParamLayout:
-    """Name -> (offset, shape) of every parameter inside the flat buffer."""
+class FlatLayout:
+    """Name -> (offset, shape) of every parameter inside one flat buffer."""
+
+    def __init__(self):
+        self.entries: Dict[str, Tuple[int, Tuple[int, ...]]] = {}
+        self.total = 0
+
+    def add(self, name: str, *shape: int) -> None:
+        self.entries[name] = (self.total, tuple(shape))
+        self.total += (math.prod(shape) + _ALIGN - 1) // _ALIGN * _ALIGN
+
+    def view(self, flat: torch.Tensor, name: str) -> torch.Tensor:
+        off, shape = self.entries[name]
+        return flat[off:off + math.prod(shape)].view(*shape)
+
+
+class ParamLayout(FlatLayout):
+    """The flat layout of a Llama-style decoder."""
 
     def __init__(self, cfg: LlamaConfig, stage: Optional[Tuple[int, int]] = None):
         """``stage = (index, n_stages)`` keeps only that pipeline stage's parameters: its block of layers, the
         embedding on the first stage, the final norm and the heads on the last (a tied LM head keeps its own
         copy of the embedding matrix on the last stage when the two stages differ)."""
+        super().__init__()
         self.cfg = cfg
-        self.entries: Dict[str, Tuple[int, Tuple[int, ...]]] = {}
         self.layer_lo, self.layer_hi = stage_layers(cfg.n_layers, stage)
         self.first = stage is None or stage[0] == 0
         self.last = stage is None or stage[0] == stage[1] - 1
-        off = 0
-
-        def add(name: str, *shape: int) -> None:
-            nonlocal off
-            self.entries[name] = (off, tuple(shape))
-            n = math.prod(shape)
-            off += (n + _ALIGN - 1) // _ALIGN * _ALIGN
-
+        add = self.add
         d, f = cfg.d_model, cfg.d_ff
         tied_head = cfg.lm_head and cfg.tie_embeddings
         if self.first or (self.last and tied_head):
@@ -139,11 +152,6 @@ class ParamLayout:
             if cfg.scalar_head:
                 add("scalar_head.w", d)
                 add("scalar_head.b", 8)  # element 0 is the bias; padded to a 16-byte slot
-        self.total = off
-
-    def view(self, flat: torch.Tensor, name: str) -> torch.Tensor:
-        off, shape = self.entries[name]
-        return flat[off:off + math.prod(shape)].view(*shape)
 
 
 @dataclass
@@ -165,6 +173,8 @@ class _FwdCtx:
 
 class LlamaModel:
     """Weights + kernels for one model instance on one GPU."""
+
+    KERNEL_SOURCES = None      # csrc files the family launches; None: the whole library
 
     def __init__(self, cfg: LlamaConfig, device, *, trainable: bool = False, recompute: str = "full",
                  weights: Optional[torch.Tensor] = None, grads: Optional[torch.Tensor] = None, seed: int = 0,

@@ -1,12 +1,16 @@
-"""Model families: Hugging Face ``config.json`` -> this engine's ``LlamaConfig``.
+"""Model families: ``config.json`` -> this engine's model configuration, and model directories -> loaded models.
 
-Two decoder families are supported, both pre-norm transformers with RMSNorm, rotary embeddings,
+Two Hugging Face decoder families (``model_type``) become a ``LlamaConfig``, both pre-norm transformers with RMSNorm, rotary embeddings,
 SwiGLU and (grouped-query) attention with head_dim 128:
 
   llama   Llama 2 / 3 (``model_type: llama``); optional llama3 rope scaling (low_freq_factor 1,
           high_freq_factor 4, original context 8192 are the only accepted parameters); optional tied
           embeddings
   qwen3   Qwen3 dense models (``model_type: qwen3``): as llama plus per-head RMSNorm on queries and keys
+
+A file that names an ``architecture`` instead lists its layers one by one:
+
+  Dulisun  chunked attention with a sink, mixtures of experts, output norms (``models/dulisun.py``); served only
 
 Anything the kernels do not implement is rejected here with a clear message (linear biases, attention
 dropout, other rope scaling types, head_dim != 128, sliding windows). Reference:
@@ -19,9 +23,11 @@ from pathlib import Path
 from typing import Any, Dict, Mapping
 
 from ..runtime.errors import RuntimeConfigError
-from .llama import LlamaConfig
+from .dulisun import AttentionMixer, DecoderLayer, DulisunConfig, DulisunModel, ExpertMixture
+from .llama import LlamaConfig, LlamaModel
 
 FAMILIES = ("llama", "qwen3")
+ARCHITECTURES = ("Dulisun",)
 
 
 def _llama3_rope_factor(cfg: Mapping[str, Any]) -> float:
@@ -42,7 +48,83 @@ def _llama3_rope_factor(cfg: Mapping[str, Any]) -> float:
     return max(1.0, float(raw.get("factor", 1.0)))
 
 
-def config_from_hf(hf: Mapping[str, Any], *, max_pos: int | None = None, lm_head: bool = True, scalar_head: bool = False) -> LlamaConfig:
+def _attention_mixer(m: Mapping[str, Any], where: str) -> AttentionMixer:
+    heads, kv, dim = int(m["heads"]), int(m["kv_heads"]), int(m["dim"])
+    rot = m.get("rot") or {}
+    rot_dims = int(rot.get("dims", 0))
+    mask = m.get("mask") or {}
+    if heads < 1 or kv < 1 or heads % kv:
+        raise RuntimeConfigError(f"{where}: {heads} query heads do not divide over {kv} key/value heads")
+    if int(m.get("vdim", dim)) != dim:
+        raise RuntimeConfigError(f"{where}: the values are the projected keys, so vdim must equal dim ({dim}), got {m['vdim']}")
+    if not 1 <= dim <= 256:
+        raise RuntimeConfigError(f"{where}: head size {dim} is not supported (the attention kernels cover 1 to 256)")
+    if rot_dims < 0 or rot_dims > dim or rot_dims % 2:
+        raise RuntimeConfigError(f"{where}: rot.dims must be even and at most dim, got {rot_dims}")
+    window = int(mask.get("size", 0))
+    if mask and window < 1:
+        raise RuntimeConfigError(f"{where}: mask.size must be at least 1")
+    return AttentionMixer(heads=heads, kv_heads=kv, dim=dim, scale=float(m["scale"]), window=window, rot_dims=rot_dims,
+                          rot_base=float(rot.get("base", 10000.0)))
+
+
+def _expert_mixture(m: Mapping[str, Any], where: str) -> ExpertMixture:
+    if m.get("kind", "moe") != "moe":
+        raise RuntimeConfigError(f"{where}: unsupported feed-forward kind {m['kind']!r}; only moe is implemented")
+    r = m["router"]
+    groups = r.get("groups") or {"count": 1, "keep": 1}
+    shared = m.get("shared") or {}
+    e = ExpertMixture(experts=int(r["experts"]), top=int(r["top"]), ff=int(m["expert"]["ff"]), shared_ff=int(shared.get("ff", 0)),
+                      groups=int(groups["count"]), keep=int(groups["keep"]))
+    if e.experts < 1 or e.ff < 1 or e.groups < 1 or e.experts % e.groups or not 1 <= e.keep <= e.groups:
+        raise RuntimeConfigError(f"{where}: {e.experts} experts do not form {e.groups} equal groups of which {e.keep} are kept")
+    if not 1 <= e.top <= e.keep * (e.experts // e.groups):
+        raise RuntimeConfigError(f"{where}: cannot choose {e.top} experts from {e.keep} groups of {e.experts // e.groups}")
+    if e.segments > 1024:
+        raise RuntimeConfigError(f"{where}: {e.segments} expert segments exceed the kernels' limit of 1024")
+    return e
+
+
+def dulisun_config(cfg: Mapping[str, Any], max_pos: int | None = None) -> DulisunConfig:
+    layers = []
+    for i, l in enumerate(cfg["layers"]):
+        if l.get("type") != "attention":
+            raise RuntimeConfigError(f"layer {i}: unsupported mixer type {l.get('type')!r}; only attention is implemented")
+        mlp = l.get("mlp")
+        layers.append(DecoderLayer(_attention_mixer(l["mixer"], f"layer {i} mixer"),
+                                   None if mlp is None else _expert_mixture(mlp, f"layer {i} mlp")))
+    if not layers:
+        raise RuntimeConfigError("the model has no layers")
+    return DulisunConfig(width=int(cfg["width"]), vocab=int(cfg["vocab"]), layers=tuple(layers), norm_eps=float(cfg["norm"]["eps"]),
+                         max_pos=int(max_pos or 4096))
+
+
+def dulisun_config_dict(cfg: DulisunConfig) -> Dict[str, Any]:
+    """The inverse of ``dulisun_config``."""
+    layers = []
+    for l in cfg.layers:
+        m, e = l.mixer, l.mlp
+        mixer: Dict[str, Any] = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.dim, "scale": m.scale}
+        if m.window:
+            mixer["mask"] = {"size": m.window}
+        if m.rot_dims:
+            mixer["rot"] = {"base": m.rot_base, "dims": m.rot_dims}
+        mlp: Dict[str, Any] | None = None
+        if e is not None:
+            mlp = {"kind": "moe", "expert": {"ff": e.ff}, "router": {"experts": e.experts, "top": e.top, "groups": {"count": e.groups, "keep": e.keep}}}
+            if e.shared_ff:
+                mlp["shared"] = {"ff": e.shared_ff}
+        layers.append({"type": "attention", "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Dulisun", "vocab": cfg.vocab, "width": cfg.width, "norm": {"eps": cfg.norm_eps}, "layers": layers}
+
+
+def config_from_hf(hf: Mapping[str, Any], *, max_pos: int | None = None, lm_head: bool = True, scalar_head: bool = False) -> LlamaConfig | DulisunConfig:
+    if "architecture" in hf:
+        if hf["architecture"] not in ARCHITECTURES:
+            raise RuntimeConfigError(f"unsupported architecture {hf['architecture']!r}; supported: {', '.join(ARCHITECTURES)}")
+        if scalar_head or not lm_head:
+            raise RuntimeConfigError(f"{hf['architecture']} models have a language-model head only")
+        return dulisun_config(hf, max_pos)
     family = hf.get("model_type")
     if family not in FAMILIES:
         raise RuntimeConfigError(f"unsupported model_type {family!r}; supported: {', '.join(FAMILIES)}")
@@ -69,7 +151,7 @@ def config_from_hf(hf: Mapping[str, Any], *, max_pos: int | None = None, lm_head
         rope_scaling_factor=_llama3_rope_factor(hf) if family == "llama" else 1.0, family=family)
 
 
-def config_from_hf_path(path, **kw) -> LlamaConfig:
+def config_from_hf_path(path, **kw) -> LlamaConfig | DulisunConfig:
     p = Path(path)
     cfg_file = p / "config.json" if p.is_dir() else p
     if not cfg_file.exists():
@@ -77,8 +159,34 @@ def config_from_hf_path(path, **kw) -> LlamaConfig:
     return config_from_hf(json.loads(cfg_file.read_text()), **kw)
 
 
-def hf_config_dict(cfg: LlamaConfig) -> Dict[str, Any]:
+def model_class(cfg):
+    """The model class that runs a configuration."""
+    return DulisunModel if isinstance(cfg, DulisunConfig) else LlamaModel
+
+
+def load_model(path, device, *, dtype=None, max_pos: int | None = None):
+    """Build the model a directory describes (``config.json`` chooses the class) and load its weights. ``dtype``: bfloat16
+    (default) or, for families that run in it, float32. Compiles the family's kernels if they are not built yet."""
+    import torch
+
+    from ..ops import _lib
+    from ..runtime.hf import load_weights
+    cfg = config_from_hf_path(path, max_pos=max_pos)
+    cls = model_class(cfg)
+    dtype = dtype or torch.bfloat16
+    if cls is LlamaModel and dtype != torch.bfloat16:
+        raise RuntimeConfigError(f"{cfg.family} models run in bfloat16 only")
+    if torch.device(device).type == "cuda":
+        _lib.ensure(cls.KERNEL_SOURCES)
+    model = cls(cfg, device, dtype=dtype, seed=None) if cls is DulisunModel else cls(cfg, device)
+    load_weights(model, path)
+    return model
+
+
+def hf_config_dict(cfg) -> Dict[str, Any]:
     """The inverse mapping (used when exporting a checkpoint next to its architecture)."""
+    if isinstance(cfg, DulisunConfig):
+        return dulisun_config_dict(cfg)
     out: Dict[str, Any] = {
         "model_type": cfg.family, "hidden_size": cfg.d_model, "intermediate_size": cfg.d_ff, "num_hidden_layers": cfg.n_layers,
         "num_attention_heads": cfg.n_heads, "num_key_value_heads": cfg.n_kv_heads, "head_dim": cfg.head_dim, "vocab_size": cfg.vocab,

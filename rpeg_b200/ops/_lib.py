@@ -82,6 +82,17 @@ _SIGNATURES = {
     "rpeg_gather_rows": [P, P, P, I, I, P],
     "rpeg_scatter_rows": [P, P, P, I, I, I, P],
     "rpeg_splitk_reduce": [P, P, I, I, I, I, P],
+    "rpeg_sample_f32": [P, I, I, I, F, I, c_ulonglong, P, P, P, P, P],
+    "rpeg_sample_filtered_f32": [P, I, I, I, F, I, F, c_ulonglong, P, P, P, P, P],
+    "rpeg_residual_norm": [I, P, I, LL, I, P, P, I, I, LL, P, P, P, P, I, I, I, F, F, I, I, P],
+    "rpeg_rotary_append": [P, I, LL, I, I, I, I, P, P, P, P, P, I, P, I, P, P, I, I, I, I, I, I, I, F, I, P],
+    "rpeg_rows_attn": [P, I, P, P, P, I, P, P, P, P, P, I, P, P, I, I, I, I, I, I, F, I, P, P],
+    "rpeg_window_prefill": [P, I, P, P, LL, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P],
+    "rpeg_moe_route": [P, I, LL, I, I, I, I, I, I, I, P, P, P, P, P],
+    "rpeg_moe_dispatch": [P, I, P, P, P, I, I, I, P, P, P, I, P],
+    "rpeg_moe_gemm": [P, LL, P, P, P, P, I, I, I, LL, I, I, I, I, I, I, I, I, P, P],
+    "rpeg_moe_gemm_f32": [P, P, P, P, P, I, I, I, I, I, I, I, I, I, P],
+    "rpeg_gemm_f32": [P, P, P, I, I, I, I, I, I, P],
     "rpeg_flash_attn_fwd": [P, I, I, I, I, P, I, I, I, I, I, I, F, P, P, P, P],
     "rpeg_flash_attn_bwd": [P, I, I, I, I, P, P, P, P, I, I, I, I, I, I, F, P, P, P, I, P, P],
 }
@@ -89,6 +100,15 @@ _SIGNATURES = {
 
 def lib_path() -> Path:
     return _LIB_PATH
+
+
+def ensure(sources=None) -> None:
+    """Make sure a library with the kernels of the named ``csrc`` files is built and is the one ``lib()`` loads (nothing
+    happens once a library is loaded)."""
+    global _LIB_PATH
+    if _lib is None:
+        from .. import build_ext
+        _LIB_PATH = build_ext.ensure(sources)
 
 
 def lib() -> ctypes.CDLL:
@@ -110,6 +130,9 @@ def lib() -> ctypes.CDLL:
         if hasattr(handle, "rpeg_decode_attn_scratch_bytes"):
             handle.rpeg_decode_attn_scratch_bytes.argtypes = [I, I, I]
             handle.rpeg_decode_attn_scratch_bytes.restype = c_longlong
+        if hasattr(handle, "rpeg_rows_attn_scratch"):
+            handle.rpeg_rows_attn_scratch.argtypes = [I, I, I, I]
+            handle.rpeg_rows_attn_scratch.restype = c_longlong
         _lib = handle
     return _lib
 

@@ -372,12 +372,15 @@ def sample(logits: torch.Tensor, temperature: float, greedy: bool, seed: int, fo
     B, V = logits.shape
     tok = torch.empty(B, dtype=torch.int32, device=logits.device) if token_out is None else token_out
     lp = torch.empty(B, dtype=torch.float32, device=logits.device) if logp_out is None else logp_out
+    if logits.dtype not in (torch.bfloat16, torch.float32):
+        raise TypeError(f"sample: logits must be bf16 or fp32, got {logits.dtype}")
+    f32 = logits.dtype == torch.float32
     if not greedy and (0 < top_k < V or top_p < 1.0):
-        check(lib().rpeg_sample_filtered(logits.data_ptr(), B, V, logits.stride(0), temperature, int(top_k), float(top_p),
+        check((lib().rpeg_sample_filtered_f32 if f32 else lib().rpeg_sample_filtered)(logits.data_ptr(), B, V, logits.stride(0), temperature, int(top_k), float(top_p),
                                          seed & 0xFFFFFFFFFFFFFFFF, _ptr(seed_offset), _ptr(forced), tok.data_ptr(), lp.data_ptr(),
                                          _stream()), "rpeg_sample_filtered")
         return tok, lp
-    check(lib().rpeg_sample(logits.data_ptr(), B, V, logits.stride(0), temperature, int(greedy),
+    check((lib().rpeg_sample_f32 if f32 else lib().rpeg_sample)(logits.data_ptr(), B, V, logits.stride(0), temperature, int(greedy),
                             seed & 0xFFFFFFFFFFFFFFFF, _ptr(seed_offset), _ptr(forced), tok.data_ptr(), lp.data_ptr(),
                             _stream()),
           "rpeg_sample")
@@ -614,6 +617,8 @@ def decode_advance(sampled, sampled_lp, token, pos, seq_len, active, gen_count, 
 def gather_rows(x: torch.Tensor, rows: torch.Tensor) -> torch.Tensor:
     if _chk.active():
         _chk.row_indices("rpeg_gather_rows", rows, x.shape[0])
+    if x.dtype == torch.float32:                 # the kernel moves 16-bit elements: an fp32 row is a row of twice the width
+        return gather_rows(x.view(torch.bfloat16), rows).view(torch.float32)
     out = torch.empty((rows.numel(), x.shape[1]), dtype=x.dtype, device=x.device)
     check(lib().rpeg_gather_rows(x.data_ptr(), rows.data_ptr(), out.data_ptr(), rows.numel(), x.shape[1], _stream()),
           "rpeg_gather_rows")
@@ -625,3 +630,210 @@ def scatter_rows_(x: torch.Tensor, rows: torch.Tensor, src: torch.Tensor, overwr
         _chk.row_indices("rpeg_scatter_rows", rows, x.shape[0])
     check(lib().rpeg_scatter_rows(x.data_ptr(), rows.data_ptr(), src.data_ptr(), rows.numel(), x.shape[1],
                                   int(overwrite), _stream()), "rpeg_scatter_rows")
+
+
+# --------------------------------------------------------------------------- fp32 matrix products
+def gemm_f32(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
+    """``a [M, K] @ b [N, K].T`` in true fp32 (CUDA cores, no reduced-precision matrix mode)."""
+    _req(a, torch.float32, "a")
+    _req(b, torch.float32, "b")
+    if a.dim() != 2 or b.dim() != 2 or a.stride(1) != 1 or b.stride(1) != 1 or a.shape[1] != b.shape[1]:
+        raise ValueError("gemm_f32 operands must be [M, K] and [N, K] with a contiguous last dimension")
+    M, Kd = a.shape
+    N = b.shape[0]
+    if out is None:
+        out = torch.empty((M, N), dtype=torch.float32, device=a.device)
+    check(lib().rpeg_gemm_f32(a.data_ptr(), b.data_ptr(), out.data_ptr(), M, N, Kd, a.stride(0), b.stride(0), out.stride(0), _stream()),
+          "rpeg_gemm_f32")
+    return out
+
+
+# --------------------------------------------------------------------------- norms around an fp32 residual stream
+_NORM_ACT, _NORM_PARTIALS, _NORM_MOE, _NORM_EMBED, _NORM_STREAM = range(5)
+
+
+class MoEOutput:
+    """Expert outputs of ``T`` tokens before their weighted sum: ``y`` rows in segment order, ``row_of`` / ``weights`` ``[T, top]``."""
+
+    __slots__ = ("y", "row_of", "weights", "top", "n_shared")
+
+    def __init__(self, y: torch.Tensor, row_of: torch.Tensor, weights: torch.Tensor, n_shared: int):
+        self.y, self.row_of, self.weights, self.n_shared = y, row_of, weights, n_shared
+        self.top = row_of.shape[1]
+
+
+def residual_norm(src, w: torch.Tensor, eps: float, d: int, *, x: torch.Tensor | None = None, add: bool = True, ids: torch.Tensor | None = None,
+                  w2: torch.Tensor | None = None, want_act: bool = True, zero_centered: bool = True) -> torch.Tensor | None:
+    """``v = norm(src)``; with ``add`` the fp32 stream ``x [T, dp]`` becomes ``x + v``, without it ``x`` (if given) becomes
+    ``v``. ``src``: an activation ``[T, >= dp]``, ``Partials``, ``MoEOutput``, an embedding table (with ``ids``) or the stream
+    itself (fp32, when the weights are bf16). Norm weights (their dtype is the activation dtype) are applied as
+    ``1 + w`` when ``zero_centered``; the mean runs over the first ``d`` of the padded ``dp = w.numel()`` columns.
+    Returns the result in the activation dtype, or, with ``w2``, ``norm(result)`` under the weight ``w2``."""
+    dp = w.numel()
+    f32 = w.dtype == torch.float32
+    splits, stride, idx, wts, top, n_shared, shared0 = 1, 0, None, None, 0, 0, 0
+    if isinstance(src, Partials):
+        kind, rows, ld, p, splits, stride = _NORM_PARTIALS, src.M, src.N, src.buf, src.splits, src.stride
+    elif isinstance(src, MoEOutput):
+        kind, p, ld, rows = _NORM_MOE, src.y, src.y.stride(0), src.row_of.shape[0]
+        idx, wts, top, n_shared, shared0 = src.row_of, src.weights, src.top, src.n_shared, rows * src.top
+    elif ids is not None:
+        _req(ids, torch.int32, "ids")
+        if _chk.active():
+            _chk.embed("rpeg_residual_norm", ids, src.shape[0])
+        kind, p, ld, rows, idx = _NORM_EMBED, src, src.stride(0), ids.numel(), ids
+    else:
+        kind, p, ld, rows = (_NORM_STREAM if src.dtype == torch.float32 and not f32 else _NORM_ACT), src, src.stride(0), src.shape[0]
+        if src.dtype not in (torch.float32, w.dtype):
+            raise TypeError(f"residual_norm: source dtype {src.dtype} does not go with weights of {w.dtype}")
+    if ld < dp or (add and x is None) or (x is not None and (x.dtype != torch.float32 or x.shape != (rows, dp) or not x.is_contiguous())):
+        raise ValueError("residual_norm: the stream must be a contiguous fp32 [T, dp] tensor and the source at least dp wide")
+    y = torch.empty((rows, dp), dtype=w.dtype, device=w.device) if (want_act or w2 is not None) else None
+    check(lib().rpeg_residual_norm(kind, p.data_ptr(), splits, stride, ld, _ptr(idx), _ptr(wts), top, n_shared, shared0, w.data_ptr(), _ptr(w2),
+                                   _ptr(x), _ptr(y), rows, d, dp, eps, 1.0 if zero_centered else 0.0, int(add), int(f32), _stream()),
+          "rpeg_residual_norm")
+    return y
+
+
+# --------------------------------------------------------------------------- chunked attention with a sink
+def rotary_append(src, q_out: torch.Tensor, q_col0: int, k_col0: int, v_col0: int, slot, pos, cos_t, sin_t, page_table, kcache, vcache,
+                  n_heads: int, dim: int, rot_dims: int, norm_eps: float | None) -> None:
+    """Interleaved rotary embedding of the first ``rot_dims`` dimensions of the q and k heads of ``src`` (an activation or
+    ``Partials``), then (``norm_eps`` not None) a weight-free RMS norm over ``dim`` per head; q goes to ``q_out``, k and the
+    values (columns from ``v_col0``, as projected) to the cache ``[pages, n_kv, PAGE, dp]``. ``v_col0 == k_col0``: the values
+    are the keys' projection."""
+    n_kv, dp = kcache.shape[1], kcache.shape[3]
+    part = isinstance(src, Partials)
+    rows, ld = (src.M, src.N) if part else (src.shape[0], src.stride(0))
+    f32 = kcache.dtype == torch.float32
+    if part and f32:
+        raise TypeError("rotary_append: split-K partials belong to the bf16 path")
+    if q_out.dtype != kcache.dtype or vcache.dtype != kcache.dtype or (not part and src.dtype != kcache.dtype):
+        raise TypeError("rotary_append: source, query buffer and caches must share a dtype")
+    if rot_dims and (cos_t.shape[1] * 2 != rot_dims or cos_t.shape != sin_t.shape):
+        raise ValueError("rotary_append: the tables do not fit rot_dims")
+    if _chk.active():
+        _chk.kv_append("rpeg_rotary_append", rows, slot, pos, page_table, kcache, n_kv, dp, cos_t if rot_dims else None)
+    check(lib().rpeg_rotary_append((src.buf if part else src).data_ptr(), src.splits if part else 0, src.stride if part else 0, ld, q_col0, k_col0,
+                                   v_col0, slot.data_ptr(), pos.data_ptr(), _ptr(cos_t), _ptr(sin_t), page_table.data_ptr(),
+                                   page_table.stride(0), q_out.data_ptr(), q_out.stride(0), kcache.data_ptr(), vcache.data_ptr(), rows, n_heads,
+                                   n_kv, dim, dp, rot_dims, int(norm_eps is not None), 0.0 if norm_eps is None else norm_eps, int(f32), _stream()),
+          "rpeg_rotary_append")
+
+
+def rows_attn_scratch(rows: int, n_heads: int, dp: int, nsplit: int) -> int:
+    """fp32 elements of split scratch ``rows_attn`` needs."""
+    return int(lib().rpeg_rows_attn_scratch(rows, n_heads, dp, nsplit))
+
+
+def rows_attn(q: torch.Tensor, kcache, vcache, page_table, slot, pos, n_heads: int, *, window: int = 0, scale: float, lens=None,
+              sink: torch.Tensor | None = None, nsplit: int = 1, scratch: torch.Tensor | None = None,
+              arrive: torch.Tensor | None = None) -> torch.Tensor:
+    """One query row per token over the paged cache: row ``t`` sees keys ``[floor(p / window) * window, p]`` of page-table row
+    ``slot[t]`` with ``p = pos[t]`` (or ``lens[t] - 1``; ``lens[t] = 0``: nothing, the row is zero). ``sink [H]`` fp32 joins the
+    softmax denominator. ``nsplit > 1`` needs ``scratch`` (see ``rows_attn_scratch``) and ``arrive`` (int32 ``rows * H``, zero)."""
+    n_kv, dp = kcache.shape[1], kcache.shape[3]
+    rows = q.shape[0]
+    if q.dtype != kcache.dtype:
+        raise TypeError("rows_attn: q and the caches must share a dtype")
+    if _chk.active():
+        seen = (pos + 1) if lens is None else lens
+        _chk.paged_attention("rpeg_rows_attn", rows, seen, page_table[slot[:rows].long()], kcache, n_kv, dp)
+    if nsplit > 1 and (scratch is None or scratch.numel() < rows_attn_scratch(rows, n_heads, dp, nsplit) or arrive is None or arrive.numel() < rows * n_heads):
+        raise ValueError("rows_attn: split attention needs scratch and arrival counters")
+    out = torch.empty((rows, n_heads * dp), dtype=q.dtype, device=q.device)
+    check(lib().rpeg_rows_attn(q.data_ptr(), q.stride(0), kcache.data_ptr(), vcache.data_ptr(), page_table.data_ptr(), page_table.stride(0),
+                               slot.data_ptr(), pos.data_ptr(), _ptr(lens), _ptr(sink), out.data_ptr(), out.stride(0), _ptr(scratch), _ptr(arrive),
+                               rows, n_heads, n_kv, dp, window, nsplit, scale, int(q.dtype == torch.float32), status_word(q.device).data_ptr(),
+                               _stream()), "rpeg_rows_attn")
+    return out
+
+
+WINDOW_PREFILL_MAX_DIM = 128     # head sizes the tensor-core prompt kernel covers
+
+
+def window_prefill(q: torch.Tensor, kcache, vcache, page_table, cu, pos, slot, max_len: int, n_heads: int, *, window: int = 0, scale: float,
+                   sink: torch.Tensor | None = None) -> torch.Tensor:
+    """Prompt attention of packed portions (request ``b`` owns rows ``cu[b] .. cu[b + 1]`` at consecutive positions) over the
+    paged cache that already holds their keys; visibility as in ``rows_attn``. bf16, head size up to 128, ``scale > 0``."""
+    _req(q, torch.bfloat16, "q")
+    n_kv, dp = kcache.shape[1], kcache.shape[3]
+    T = q.shape[0]
+    if _chk.active():
+        _chk.packed_sequences("rpeg_window_prefill", cu, T, max_len)
+        _chk.paged_attention("rpeg_window_prefill", T, pos + 1, page_table[slot[:T].long()], kcache, n_kv, dp)
+    out = torch.empty((T, n_heads * dp), dtype=torch.bfloat16, device=q.device)
+    check(lib().rpeg_window_prefill(q.data_ptr(), q.stride(0), kcache.data_ptr(), vcache.data_ptr(), kcache.shape[0], page_table.data_ptr(),
+                                    page_table.stride(0), cu.data_ptr(), pos.data_ptr(), slot.data_ptr(), _ptr(sink), out.data_ptr(),
+                                    out.stride(0), T, cu.numel() - 1, max_len, n_heads, n_kv, dp, window, scale,
+                                    status_word(q.device).data_ptr(), _stream()), "rpeg_window_prefill")
+    return out
+
+
+# --------------------------------------------------------------------------- mixture of experts
+class MoERouting:
+    """Where the tokens of one mixture layer go: ``ids`` / ``weights`` / ``row_of`` ``[T, top]``, ``seg_off [E + 1]`` and the
+    dispatched rows ``x_sorted [T * top, dp]``."""
+
+    __slots__ = ("ids", "weights", "row_of", "seg_off", "x_sorted", "x")
+
+    def __init__(self, ids, weights, row_of, seg_off, x_sorted, x):
+        self.ids, self.weights, self.row_of, self.seg_off, self.x_sorted, self.x = ids, weights, row_of, seg_off, x_sorted, x
+
+
+def moe_route(logits, n_experts: int, top: int, counts: torch.Tensor, *, n_groups: int = 1, keep_groups: int = 1, renormalize: bool = False):
+    """Softmax routing of ``logits`` (fp32 ``[T, >= E]`` or ``Partials``): the ``top`` largest scores among the experts of the
+    ``keep_groups`` best of ``n_groups`` equal groups. ``counts [E]`` int32 must be zero; every choice takes a ticket there.
+    Returns ``(ids, weights, tickets)``, each ``[T, top]``."""
+    part = isinstance(logits, Partials)
+    rows, ld = (logits.M, logits.N) if part else (logits.shape[0], logits.stride(0))
+    buf = logits.buf if part else logits
+    _req(buf, torch.float32, "router logits")
+    if counts.numel() < n_experts or ld < n_experts:
+        raise ValueError("moe_route: counts and logits must cover every expert")
+    i32 = dict(dtype=torch.int32, device=buf.device)
+    ids, ticket = torch.empty((rows, top), **i32), torch.empty((rows, top), **i32)
+    wts = torch.empty((rows, top), dtype=torch.float32, device=buf.device)
+    check(lib().rpeg_moe_route(buf.data_ptr(), logits.splits if part else 1, logits.stride if part else 0, ld, rows, n_experts, n_groups, keep_groups,
+                               top, int(renormalize), ids.data_ptr(), wts.data_ptr(), ticket.data_ptr(), counts.data_ptr(), _stream()),
+          "rpeg_moe_route")
+    return ids, wts, ticket
+
+
+def moe_dispatch(x: torch.Tensor, ids, wts, ticket, counts, n_experts: int) -> MoERouting:
+    """Copy every token's row into the segments of its experts."""
+    rows, dp = x.shape
+    top = ids.shape[1]
+    if not x.is_contiguous():
+        raise ValueError("moe_dispatch: the rows must be contiguous")
+    row_of = torch.empty_like(ids)
+    seg_off = torch.empty(n_experts + 1, dtype=torch.int32, device=x.device)
+    xs = torch.empty((rows * top, dp), dtype=x.dtype, device=x.device)
+    check(lib().rpeg_moe_dispatch(x.data_ptr(), dp, ids.data_ptr(), ticket.data_ptr(), counts.data_ptr(), rows, n_experts, top, xs.data_ptr(),
+                                  row_of.data_ptr(), seg_off.data_ptr(), int(x.dtype == torch.float32), _stream()), "rpeg_moe_dispatch")
+    return MoERouting(ids, wts, row_of, seg_off, xs, x)
+
+
+def moe_gemm(a: torch.Tensor, b: torch.Tensor, r: MoERouting, n_experts: int, n_shared: int, *, shared_x: torch.Tensor | None = None,
+             gelu: bool = False, bn: int = 0) -> torch.Tensor:
+    """``C[rows of segment s] = act(a[rows of s] @ b[s].T)`` over the experts' segments; ``b [E + n_shared, N, K]``. The always-on
+    segments take their rows from ``shared_x [T, K]`` (tokens in order) or, without it, from ``a`` behind the routed rows."""
+    T, top = r.row_of.shape
+    S, N, Kd = b.shape
+    if S != n_experts + n_shared or a.shape[1] != Kd or not b.is_contiguous() or a.stride(1) != 1:
+        raise ValueError("moe_gemm: operand shapes do not fit the segments")
+    need = T * top + (0 if shared_x is not None else n_shared * T)
+    if a.shape[0] < need or (shared_x is not None and (shared_x.shape != (T, Kd) or shared_x.stride(1) != 1)):
+        raise ValueError("moe_gemm: too few operand rows")
+    c = torch.empty((T * (top + n_shared), N), dtype=a.dtype, device=a.device)
+    if a.dtype == torch.float32:
+        if shared_x is not None and shared_x.stride(0) != a.stride(0):
+            raise ValueError("moe_gemm: both operands need one row pitch")
+        check(lib().rpeg_moe_gemm_f32(a.data_ptr(), _ptr(shared_x), b.data_ptr(), c.data_ptr(), r.seg_off.data_ptr(), n_experts, n_shared, T, N, Kd,
+                                      a.stride(0), Kd, c.stride(0), int(gelu), _stream()), "rpeg_moe_gemm_f32")
+        return c
+    _req(a, torch.bfloat16, "a")
+    check(lib().rpeg_moe_gemm(a.data_ptr(), a.shape[0], _ptr(shared_x), b.data_ptr(), c.data_ptr(), r.seg_off.data_ptr(), n_experts, n_shared, T,
+                              T * top, N, Kd, a.stride(0), 0 if shared_x is None else shared_x.stride(0), Kd, c.stride(0), int(gelu), bn,
+                              status_word(a.device).data_ptr(), _stream()), "rpeg_moe_gemm")
+    return c

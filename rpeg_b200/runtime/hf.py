@@ -12,6 +12,7 @@ from __future__ import annotations
 import json
 import re
 import struct
+import warnings
 from pathlib import Path
 from typing import Any, Dict, Iterable, Optional, Tuple
 
@@ -151,6 +152,54 @@ def load_hf_weights(model, model_dir) -> int:
     if cfg.lm_head and not cfg.tie_embeddings:
         put(model.p["lm_head"], get("lm_head.weight" if "lm_head.weight" in idx else "model.embed_tokens.weight"))
     return copied
+
+
+def load_dulisun_weights(model, model_dir) -> int:
+    """Copy a Dulisun checkpoint into ``model``: linear weights are ``[out, in]`` under ``l<i>.mix.*`` and ``l<i>.mlp.*``,
+    queries and keys are stacked, experts become the segments of one grouped matrix. Tensors without a place are reported
+    as a warning. Returns the number of parameters copied."""
+    cfg = model.cfg
+    idx = _open_shards(model_dir)
+    used = set()
+    copied = 0
+
+    def get(name: str, *shape: int):
+        nonlocal copied
+        if name not in idx:
+            raise RuntimeConfigError(f"tensor {name} is missing from {model_dir}")
+        t = idx[name].get_tensor(name)
+        if tuple(t.shape) != shape:
+            raise RuntimeConfigError(f"shape mismatch of {name}: checkpoint {tuple(t.shape)} vs model {shape}")
+        used.add(name)
+        copied += t.numel()
+        return t.to(device=model.device, dtype=model.dtype)
+
+    d = cfg.width
+    model.p["embed"][: cfg.vocab, :d].copy_(get("embed", cfg.vocab, d))
+    model.p["embed_norm"][:d].copy_(get("embed.norm", d))
+    model.p["final_norm"][:d].copy_(get("final.norm", d))
+    for i, layer in enumerate(cfg.layers):
+        m, e = layer.mixer, layer.mlp
+        model.put_qk(i, get(f"l{i}.mix.q", m.heads * m.dim, d), get(f"l{i}.mix.k", m.kv_heads * m.dim, d))
+        model.put_o(i, get(f"l{i}.mix.o", d, m.heads * m.dim))
+        model.sink[i].copy_(get(f"l{i}.mix.sink", m.heads).float())
+        model.p[f"l{i}.norm1"][:d].copy_(get(f"l{i}.norm1", d))
+        if e is not None:
+            model.p[f"l{i}.router"][: e.experts, :d].copy_(get(f"l{i}.mlp.router", e.experts, d))
+            for s in range(e.experts):
+                model.put_expert(i, s, get(f"l{i}.mlp.e{s}.up", e.ff, d), get(f"l{i}.mlp.e{s}.down", d, e.ff))
+            if e.shared_ff:
+                model.put_shared(i, get(f"l{i}.mlp.shared.up", e.shared_ff, d), get(f"l{i}.mlp.shared.down", d, e.shared_ff))
+            model.p[f"l{i}.norm2"][:d].copy_(get(f"l{i}.norm2", d))
+    left = sorted(set(idx) - used)
+    if left:
+        warnings.warn(f"{model_dir} holds {len(left)} tensors this model has no place for: {', '.join(left[:5])}", stacklevel=2)
+    return copied
+
+
+def load_weights(model, model_dir) -> int:
+    """Load a checkpoint with the naming of the model's family."""
+    return (load_dulisun_weights if getattr(model.cfg, "family", "") == "dulisun" else load_hf_weights)(model, model_dir)
 
 
 def save_hf_weights(model, model_dir, shard_bytes: int = 4 << 30) -> None:
