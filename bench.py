@@ -11,6 +11,8 @@ sampled generation up to 2048 tokens with EOS forced at lengths drawn from the q
 [0.5 -> 512, 0.9 -> 1024, 1.0 -> 2048], rewards ~ N(0,1) group-normalised, bf16 compute, fp32 Adam.
 The total batch is fixed, so more GPUs means strong scaling (data parallel over prompts).
 
+``--serve`` replaces the workload by a serving comparison (``rpeg_b200/engine/serve_bench.py``) and prints its own line.
+
 Rank 0 prints ONE JSON line. ``value`` is samples/s over all GPUs from CUDA-event timing of K steps
 whose inputs already sit on the device; ``e2e`` repeats K steps through the public ``step`` API with
 pinned host inputs (H2D copy) and the loss read back (D2H). ``--impl reference`` reports why the
@@ -223,6 +225,8 @@ def main() -> None:
                          "tcgen05 kernel) instead of once per row through L2; off by default: measured slower on the full step")
     ap.add_argument("--budget-s", type=float, default=420.0,
                     help="wall-clock budget for warm-up plus timed steps; the timed step count is cut to fit and reported")
+    ap.add_argument("--serve", action="store_true", help="instead of the RLHF iteration: prefill and decode throughput of the Dulisun family "
+                    "beside the Llama family at equal size, with every kernel's distance from its roofline (one GPU)")
     args = ap.parse_args()
     # Libraries (NCCL's version banner, for one) write to file descriptor 1. The contract is ONE JSON line on
     # stdout, so everything else is sent to stderr and the line goes to the saved descriptor at the end.
@@ -233,6 +237,14 @@ def main() -> None:
     def emit(obj) -> None:
         sys.stdout.flush()
         os.write(real_stdout, (json.dumps(obj) + "\n").encode())
+
+    if args.serve:
+        from rpeg_b200.engine import serve_bench
+        sampler = ClockSampler(0)
+        sampler.start()
+        line = serve_bench.run(["2b", "7b"], 4)
+        emit({**line, "clocks": sampler.stop()})
+        return
 
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))

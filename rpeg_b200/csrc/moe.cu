@@ -19,19 +19,18 @@ namespace rpeg {
 constexpr int MOE_MAX_SEGMENTS = 1024;
 constexpr int ROUTE_WARPS = 4;
 
-// Index of the largest value of v[0..n) whose flag is zero, ties to the smaller index; every lane returns it (-1: none).
-__device__ __forceinline__ int warp_argmax_free(const float* v, const unsigned char* taken, int n, int lane) {
-  float best = -INFINITY;
+// Index of the largest of the non-negative values v[lane + 32 j] whose bit j is set in the lane's mask, ties to the smaller
+// index; every lane returns it (-1: no bit set anywhere). Non-negative floats order like their bit patterns.
+__device__ __forceinline__ int warp_argmax(const float* v, int n, uint32_t mask, int lane) {
+  uint32_t best = 0u;
   int at = 0x7fffffff;
-  for (int i = lane; i < n; i += 32)
-    if (!taken[i] && (v[i] > best || at == 0x7fffffff)) { best = v[i]; at = i; }
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    const float b2 = __shfl_xor_sync(0xffffffffu, best, o);
-    const int i2 = __shfl_xor_sync(0xffffffffu, at, o);
-    if (i2 != 0x7fffffff && (at == 0x7fffffff || b2 > best || (b2 == best && i2 < at))) { best = b2; at = i2; }
+  for (int j = 0, i = lane; i < n; ++j, i += 32) {
+    const uint32_t key = (mask >> j) & 1u ? __float_as_uint(v[i]) + 1u : 0u;
+    if (key > best) { best = key; at = i; }
   }
-  return at == 0x7fffffff ? -1 : at;
+  const uint32_t top = __reduce_max_sync(0xffffffffu, best);
+  if (top == 0u) return -1;
+  return static_cast<int>(__reduce_min_sync(0xffffffffu, best == top ? static_cast<uint32_t>(at) : 0x7fffffffu));
 }
 
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
@@ -42,17 +41,15 @@ moe_route_kernel(const float* __restrict__ logits, int splits, long long stride,
   extern __shared__ float route_sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * ROUTE_WARPS + warp;
-  // per warp: E scores, n_groups group scores, E + n_groups flags
-  const int words = E + n_groups + (E + n_groups + 3) / 4;
-  float* sc = route_sm + warp * words;
-  float* gs = sc + E;
-  unsigned char* taken = reinterpret_cast<unsigned char*>(gs + n_groups);
-  unsigned char* gtaken = taken + E;
   if (t >= rows) return;
+  float* sc = route_sm + warp * (E + n_groups + top);     // per warp: E scores, n_groups group scores, the choices
+  float* gs = sc + E;
+  int* pick = reinterpret_cast<int*>(gs + n_groups);
   const float* lr = logits + static_cast<size_t>(t) * ld;
   float mx = -INFINITY;
   for (int e = lane; e < E; e += 32) {
     float z = lr[e];
+#pragma unroll 8
     for (int s = 1; s < splits; ++s) z += lr[s * stride + e];
     sc[e] = z;
     mx = fmaxf(mx, z);
@@ -64,45 +61,43 @@ moe_route_kernel(const float* __restrict__ logits, int splits, long long stride,
     sc[e] = p;
     sum += p;
   }
-  sum = warp_sum(sum);
-  const float inv = 1.f / sum;
-  const int per = E / n_groups;
-  for (int e = lane; e < E; e += 32) { sc[e] *= inv; taken[e] = keep < n_groups ? 1 : 0; }
+  const float inv = 1.f / warp_sum(sum);
+  for (int e = lane; e < E; e += 32) sc[e] *= inv;
   __syncwarp();
+  const int per = E / n_groups;
+  uint32_t open = 0xffffffffu;                             // bit j: expert lane + 32 j may still be chosen (E <= 1024)
   if (keep < n_groups) {
     for (int g = lane; g < n_groups; g += 32) {
       float b = sc[g * per];
       for (int i = 1; i < per; ++i) b = fmaxf(b, sc[g * per + i]);
       gs[g] = b;
-      gtaken[g] = 0;
     }
     __syncwarp();
+    open = 0u;
+    uint32_t gopen = 0xffffffffu;
     for (int k = 0; k < keep; ++k) {
-      const int g = warp_argmax_free(gs, gtaken, n_groups, lane);
-      __syncwarp();
-      if (g >= 0) {
-        if (lane == 0) gtaken[g] = 1;
-        for (int i = lane; i < per; i += 32) taken[g * per + i] = 0;
-      }
-      __syncwarp();
+      const int g = max(warp_argmax(gs, n_groups, gopen, lane), 0);
+      if ((g & 31) == lane) gopen &= ~(1u << (g >> 5));
+      for (int j = 0, e = lane; e < E; ++j, e += 32)
+        if (e >= g * per && e < (g + 1) * per) open |= 1u << j;
     }
   }
   float chosen = 0.f;
   for (int k = 0; k < top; ++k) {
-    const int e = max(warp_argmax_free(sc, taken, E, lane), 0);      // the host guarantees top <= keep * per
-    __syncwarp();
+    const int e = max(warp_argmax(sc, E, open, lane), 0);  // the host guarantees top <= keep * per
+    if ((e & 31) == lane) open &= ~(1u << (e >> 5));
     chosen += sc[e];
-    if (lane == 0) {
-      taken[e] = 1;
-      const size_t o = static_cast<size_t>(t) * top + k;
-      ids[o] = e;
-      wts[o] = sc[e];
-      ticket[o] = atomicAdd(&counts[e], 1);
-    }
-    __syncwarp();
+    if (lane == 0) pick[k] = e;
   }
-  if (renorm && lane == 0)
-    for (int k = 0; k < top; ++k) wts[static_cast<size_t>(t) * top + k] /= chosen;
+  __syncwarp();
+  const float scale = renorm ? 1.f / chosen : 1.f;
+  for (int k = lane; k < top; k += 32) {
+    const int e = pick[k];
+    const size_t o = static_cast<size_t>(t) * top + k;
+    ids[o] = e;
+    wts[o] = sc[e] * scale;
+    ticket[o] = atomicAdd(&counts[e], 1);
+  }
 }
 
 // One CTA per token. Every CTA sums the counters below its token's experts itself (a few hundred words from L2).
@@ -377,7 +372,7 @@ extern "C" int rpeg_moe_route(const float* logits, int splits, long long stride,
   if (rows <= 0) return 0;
   if (E < 1 || n_groups < 1 || E % n_groups || keep < 1 || keep > n_groups || top < 1 || top > keep * (E / n_groups)) return -2;
   if (E > MOE_MAX_SEGMENTS) return -3;
-  const size_t smem = static_cast<size_t>(ROUTE_WARPS) * (E + n_groups + (E + n_groups + 3) / 4) * 4;
+  const size_t smem = static_cast<size_t>(ROUTE_WARPS) * (E + n_groups + top) * 4;
   if (smem > 48 * 1024) return -3;
   const cudaError_t e = launch_pdl(moe_route_kernel, dim3((rows + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem,
                                    STREAM(stream), logits, splits, stride, ld, rows, E, n_groups, keep, top, renorm, ids, wts, ticket, counts);

@@ -19,8 +19,10 @@ namespace rpeg {
 
 constexpr int WPAGE = RPEG_KV_PAGE;
 
-// One warp per (token, head): query heads, then KV heads. A lane owns whole pairs (2i, 2i + 1), so the rotation is local.
-template <typename T, bool PARTIALS>
+// One warp per HPW heads of a token (query heads, then KV heads). A lane owns runs of 4 elements, i.e. whole pairs
+// (2i, 2i + 1), so the rotation is local; a rotation keeps the sum of squares, so the norm is known before it. Prompts take
+// four heads per warp (the angles are read once for all of them), decode one (more warps for few tokens).
+template <typename T, bool PARTIALS, int HPW>
 __global__ void __launch_bounds__(256)
 rotary_append_kernel(const void* __restrict__ src_v, int splits, long long stride, int ld, int q_col0, int k_col0, int v_col0,
                      const int* __restrict__ slot, const int* __restrict__ pos, const float* __restrict__ cos_t,
@@ -29,67 +31,77 @@ rotary_append_kernel(const void* __restrict__ src_v, int splits, long long strid
                      float eps) {
   griddep_launch();
   griddep_wait();
-  const int jobs = H + Hkv;
-  const long long wid = (static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x) >> 5;
-  if (wid >= static_cast<long long>(rows) * jobs) return;
+  const unsigned jobs = (H + Hkv + HPW - 1) / HPW;
+  const unsigned wid = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);     // below 2^31, checked on the host
+  if (wid >= static_cast<unsigned>(rows) * jobs) return;
   const int lane = threadIdx.x & 31;
-  const int t = static_cast<int>(wid / jobs), job = static_cast<int>(wid % jobs);
+  const int t = static_cast<int>(wid / jobs), job0 = static_cast<int>(wid % jobs) * HPW;
   const int p = pos[t];
-  const bool is_q = job < H;
-  const int half = rot_dims >> 1, npair = dp >> 1;
-  auto read = [&](int col) -> float2 {
+  const int half = rot_dims >> 1, nq = dp >> 2;
+  auto read = [&](int col) -> float4 {
     const size_t off = static_cast<size_t>(t) * ld + col;
     if constexpr (PARTIALS) {
       const float* s = static_cast<const float*>(src_v) + off;
-      float2 a = load2(s);
-      for (int k = 1; k < splits; ++k) {
-        const float2 b = load2(s + k * stride);
-        a.x += b.x; a.y += b.y;
-      }
+      float4 a = load4(s);
+#pragma unroll 8
+      for (int k = 1; k < splits; ++k) a = add4(a, load4(s + k * stride));
       return a;
     } else {
-      return load2(static_cast<const T*>(src_v) + off);
+      return load4(static_cast<const T*>(src_v) + off);
     }
   };
-  const int hk = job - H;
-  const int col0 = is_q ? q_col0 + job * dp : k_col0 + hk * dp;
-  float2 v[4];
-  float ss = 0.f;
+  float4 v[HPW][2];
 #pragma unroll
-  for (int j = 0; j < 4; ++j) {
-    const int i = lane + 32 * j;
-    if (i < npair) {
-      v[j] = read(col0 + 2 * i);
-      ss += v[j].x * v[j].x + v[j].y * v[j].y;         // a rotation keeps the sum of squares of its pair
+  for (int g = 0; g < HPW; ++g) {
+    const int job = job0 + g;
+    const int col0 = job < H ? q_col0 + job * dp : k_col0 + (job - H) * dp;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      v[g][j] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (lane + 32 * j < nq && job < H + Hkv) v[g][j] = read(col0 + 4 * (lane + 32 * j));
     }
   }
-  const float r = do_norm ? rsqrtf(warp_sum(ss) / static_cast<float>(dim) + eps) : 1.f;
-  size_t dst = 0;
-  if (!is_q) {
-    const int page = page_table[static_cast<size_t>(slot[t]) * max_pages + p / WPAGE];
-    dst = ((static_cast<size_t>(page) * Hkv + hk) * WPAGE + (p % WPAGE)) * dp;
-  }
-  T* out = is_q ? q_out + static_cast<size_t>(t) * ldq + job * dp : kcache + dst;
+  float2 cs[2][2];                                          // (cos, sin) of the lane's two pairs
 #pragma unroll
-  for (int j = 0; j < 4; ++j) {
-    const int i = lane + 32 * j;
-    if (i >= npair) break;
-    if (!is_q) {
-      const float2 raw = v_col0 == k_col0 ? v[j] : read(v_col0 + hk * dp + 2 * i);
-      store2(vcache + dst + 2 * i, raw.x, raw.y);
+  for (int j = 0; j < 2; ++j)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int pr = 2 * (lane + 32 * j) + e;
+      cs[j][e] = pr < half ? make_float2(cos_t[static_cast<size_t>(p) * half + pr], sin_t[static_cast<size_t>(p) * half + pr])
+                           : make_float2(1.f, 0.f);
     }
-    float a = v[j].x, b = v[j].y;
-    if (i < half) {
-      const float c = cos_t[static_cast<size_t>(p) * half + i], s = sin_t[static_cast<size_t>(p) * half + i];
-      a = v[j].x * c - v[j].y * s;
-      b = v[j].y * c + v[j].x * s;
+  size_t page_row = 0;
+  if (job0 + HPW > H) page_row = static_cast<size_t>(page_table[static_cast<size_t>(slot[t]) * max_pages + p / WPAGE]) * Hkv;
+#pragma unroll
+  for (int g = 0; g < HPW; ++g) {
+    const int job = job0 + g;
+    if (job >= H + Hkv) break;
+    const bool is_q = job < H;
+    float r = 1.f;
+    if (do_norm) {
+      float ss = 0.f;
+#pragma unroll
+      for (int j = 0; j < 2; ++j) ss += v[g][j].x * v[g][j].x + v[g][j].y * v[g][j].y + v[g][j].z * v[g][j].z + v[g][j].w * v[g][j].w;
+      r = rsqrtf(warp_sum(ss) / static_cast<float>(dim) + eps);
     }
-    store2(out + 2 * i, a * r, b * r);
+    const size_t dst = is_q ? 0 : ((page_row + (job - H)) * WPAGE + (p % WPAGE)) * dp;
+    T* out = is_q ? q_out + static_cast<size_t>(t) * ldq + job * dp : kcache + dst;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int i = lane + 32 * j;
+      if (i >= nq) break;
+      const float4 u = v[g][j];
+      if (!is_q) store4(vcache + dst + 4 * i, v_col0 == k_col0 ? u : read(v_col0 + (job - H) * dp + 4 * i));
+      const float2 a = cs[j][0], b = cs[j][1];
+      store4(out + 4 * i, make_float4((u.x * a.x - u.y * a.y) * r, (u.y * a.x + u.x * a.y) * r, (u.z * b.x - u.w * b.y) * r,
+                                      (u.w * b.x + u.z * b.y) * r));
+    }
   }
 }
 
 // ---------------------------------------------------------------------------------- rows attention
-constexpr int RA_THREADS = 128, RA_HEADS = 8, RA_KEYS = 4;      // heads and keys one lane group scores together
+constexpr int RA_THREADS = 128;
+constexpr size_t RA_SMEM_TARGET = 72 * 1024;     // pages in flight per CTA: three CTAs of one SM together keep the copy rate up
 
 struct RowsAttn {
   const void* q; int ldq;
@@ -144,20 +156,23 @@ __device__ __forceinline__ void bulk_load(void* smem_dst, const void* src, uint3
 }
 
 // LPK lanes hold one key (8 dimensions each), a warp scores 32 / LPK keys side by side and RA_KEYS of them per lane
-// group in a row. The RA_KEYS x RA_HEADS partial dot products of a lane are summed across its group by a transposing
+// group in a row, for RA_HEADS query heads of the KV head (4 or 8, whichever leaves fewer idle). The RA_KEYS x RA_HEADS
+// partial dot products of a lane are summed across its group by a transposing
 // butterfly after which lane c holds the finished scores number c * VPL .. of the list (key major), so every exponential
 // is computed once; the weights go back to all lanes of the group by shuffles for P V.
-template <typename T, int LPK>
+template <typename T, int LPK, int RA_HEADS, int RA_KEYS>
 __global__ void __launch_bounds__(RA_THREADS)
 rows_attn_kernel(const RowsAttn a) {
   constexpr int GPW = 32 / LPK, NV = RA_KEYS * RA_HEADS, VPL = NV / LPK, ITERS = (WPAGE / 4) / (RA_KEYS * GPW);
   constexpr int GROUPS = 4 * GPW, WIDTH = LPK * 8;
-  static_assert(VPL >= 1 && ITERS >= 1, "lane split");
+  constexpr int HL = RA_HEADS / VPL;                    // lanes that hold the scores of one key
+  static_assert(VPL >= 1 && HL >= 1 && ITERS >= 1, "lane split");
   griddep_launch();
   griddep_wait();
   extern __shared__ __align__(128) uint8_t ra_smem[];
   __shared__ uint64_t full_bar[4];
   __shared__ int abort_word, is_last;
+  __shared__ float share[RA_HEADS][64];
   __shared__ float red_m[GROUPS][RA_HEADS], red_l[GROUPS][RA_HEADS];
   const int row = blockIdx.x, split = blockIdx.z;
   const int R = a.H / a.Hkv;                            // query heads per KV head
@@ -266,8 +281,8 @@ rows_attn_kernel(const RowsAttn a) {
         for (int i = 0; i < VPL; ++i) {
           if (!valid) v[i] = -INFINITY;
           float b = v[i];
-          b = fmaxf(b, __shfl_xor_sync(0xffffffffu, b, LPK / 4));
-          b = fmaxf(b, __shfl_xor_sync(0xffffffffu, b, LPK / 2));
+#pragma unroll
+          for (int o = HL; o < LPK; o <<= 1) b = fmaxf(b, __shfl_xor_sync(0xffffffffu, b, o));
           nm[i] = fmaxf(m[i], b);
           grew |= nm[i] > m[i];
         }
@@ -319,8 +334,8 @@ rows_attn_kernel(const RowsAttn a) {
   const int gi = warp * GPW + grp;
 #pragma unroll
   for (int i = 0; i < VPL; ++i) {
-    l[i] += __shfl_xor_sync(0xffffffffu, l[i], LPK / 4);
-    l[i] += __shfl_xor_sync(0xffffffffu, l[i], LPK / 2);
+#pragma unroll
+    for (int o = HL; o < LPK; o <<= 1) l[i] += __shfl_xor_sync(0xffffffffu, l[i], o);
     if (u_own == 0) {
       red_m[gi][c * VPL + i] = m[i];
       red_l[gi][c * VPL + i] = l[i];
@@ -373,30 +388,48 @@ rows_attn_kernel(const RowsAttn a) {
   if (!is_last) return;
   if (threadIdx.x == 0) *counter = 0;
   __threadfence();
+  const float* parts = a.partial + (static_cast<size_t>(row) * a.H + h0) * a.nsplit * (dp + 2);
+  if (warp < nh)                                        // share of every split in its head's result
+    for (int h = warp; h < nh; h += RA_THREADS / 32) {
+      const float* pp = parts + static_cast<size_t>(h) * a.nsplit * (dp + 2) + dp;
+      const float sl = sink != nullptr ? sink[h0 + h] * 1.4426950408889634f : -INFINITY;
+      float ms[2], ls[2], gm = sl;
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        const int s = lane + 32 * j;
+        ms[j] = s < a.nsplit ? __ldcg(pp + s * (dp + 2)) : -INFINITY;
+        ls[j] = s < a.nsplit ? __ldcg(pp + s * (dp + 2) + 1) : 0.f;
+        gm = fmaxf(gm, ms[j]);
+      }
+      gm = warp_max(gm);
+      float gl = 0.f;
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        ms[j] = ms[j] == -INFINITY ? 0.f : exp2f(ms[j] - gm);
+        gl += ls[j] * ms[j];
+      }
+      gl = warp_sum(gl) + (sink != nullptr ? exp2f(sl - gm) : 0.f);
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+        if (lane + 32 * j < a.nsplit) share[h][lane + 32 * j] = gl > 0.f ? ms[j] / gl : 0.f;
+    }
+  __syncthreads();
   for (int e = threadIdx.x; e < nh * dp; e += RA_THREADS) {
     const int h = e / dp, d = e % dp;
-    const float* pp = a.partial + (static_cast<size_t>(row) * a.H + h0 + h) * a.nsplit * (dp + 2);
-    const float sl = sink != nullptr ? sink[h0 + h] * 1.4426950408889634f : -INFINITY;
-    float gm = sl;
-    for (int s = 0; s < a.nsplit; ++s) gm = fmaxf(gm, __ldcg(pp + s * (dp + 2) + dp));
-    float gl = sink != nullptr ? exp2f(sl - gm) : 0.f, o = 0.f;
-    for (int s = 0; s < a.nsplit; ++s) {
-      const float ms = __ldcg(pp + s * (dp + 2) + dp);
-      const float w = ms == -INFINITY ? 0.f : exp2f(ms - gm);
-      gl += __ldcg(pp + s * (dp + 2) + dp + 1) * w;
-      o += __ldcg(pp + s * (dp + 2) + d) * w;
-    }
-    const float r = gl > 0.f ? o / gl : 0.f;
+    const float* pp = parts + static_cast<size_t>(h) * a.nsplit * (dp + 2) + d;
+    float r = 0.f;
+#pragma unroll 8
+    for (int s = 0; s < a.nsplit; ++s) r += __ldcg(pp + s * (dp + 2)) * share[h][s];
     if constexpr (sizeof(T) == 2) out[(h0 + h) * dp + d] = __float2bfloat16(r); else out[(h0 + h) * dp + d] = r;
   }
 }
 
-template <typename T, int LPK>
+template <typename T, int LPK, int HEADS, int KEYS>
 static int launch_rows_attn(RowsAttn a, int rows, cudaStream_t stream) {
-  auto kern = rows_attn_kernel<T, LPK>;
+  auto kern = rows_attn_kernel<T, LPK, HEADS, KEYS>;
   const size_t stage = static_cast<size_t>(2) * WPAGE * a.dp * sizeof(T);
-  const size_t merge = static_cast<size_t>(4 * (32 / LPK)) * RA_HEADS * LPK * 8 * 4;
-  int st = static_cast<int>((100 * 1024) / stage);
+  const size_t merge = static_cast<size_t>(4 * (32 / LPK)) * HEADS * LPK * 8 * 4;
+  int st = static_cast<int>((RA_SMEM_TARGET) / stage);
   a.stages = st < 1 ? 1 : (st > 4 ? 4 : st);
   size_t smem = a.stages * stage;
   if (smem < merge) smem = merge;
@@ -407,15 +440,22 @@ static int launch_rows_attn(RowsAttn a, int rows, cudaStream_t stream) {
     configured = smem;
   }
   const int R = a.H / a.Hkv;
-  const dim3 grid(rows, a.Hkv * ((R + RA_HEADS - 1) / RA_HEADS), a.nsplit);
+  const dim3 grid(rows, a.Hkv * ((R + HEADS - 1) / HEADS), a.nsplit);
   return launch_pdl(kern, grid, dim3(RA_THREADS), smem, stream, a) == cudaSuccess ? 0 : -21;
 }
 
 template <typename T>
 static int dispatch_rows_attn(const RowsAttn& a, int rows, cudaStream_t stream) {
-  if (a.dp <= 64) return launch_rows_attn<T, 8>(a, rows, stream);
-  if (a.dp <= 128) return launch_rows_attn<T, 16>(a, rows, stream);
-  return launch_rows_attn<T, 32>(a, rows, stream);
+  const int R = a.H / a.Hkv;
+  const bool narrow = (R - 1) % 8 < 4 && R <= 12;            // blocks of 4 heads leave fewer idle
+  if (narrow) {
+    if (a.dp <= 64) return launch_rows_attn<T, 8, 4, 4>(a, rows, stream);
+    if (a.dp <= 128) return launch_rows_attn<T, 16, 4, 8>(a, rows, stream);
+    return launch_rows_attn<T, 32, 4, 8>(a, rows, stream);
+  }
+  if (a.dp <= 64) return launch_rows_attn<T, 8, 8, 4>(a, rows, stream);
+  if (a.dp <= 128) return launch_rows_attn<T, 16, 8, 4>(a, rows, stream);
+  return launch_rows_attn<T, 32, 8, 4>(a, rows, stream);
 }
 
 }  // namespace rpeg
@@ -428,17 +468,20 @@ extern "C" int rpeg_rotary_append(const void* src, int splits, long long stride,
                                   int ldq, void* kcache, void* vcache, int rows, int H, int Hkv, int dim, int dp, int rot_dims, int do_norm,
                                   float eps, int f32, void* stream) {
   if (rows <= 0) return 0;
-  if ((dp & 7) || dp > 256 || dim < 1 || dim > dp || rot_dims < 0 || rot_dims > dim || (rot_dims & 1) || ((ld | ldq) & 1)) return -2;
+  if ((dp & 7) || dp > 256 || dim < 1 || dim > dp || rot_dims < 0 || rot_dims > dim || (rot_dims & 1) || ((ld | ldq | q_col0 | k_col0 | v_col0) & 3)) return -2;
   if (H < 1 || Hkv < 1 || H % Hkv) return -3;
-  const long long warps = static_cast<long long>(rows) * (H + Hkv);
+  const int hpw = rows >= 1024 && !f32 && splits == 0 ? 4 : 1;
+  const long long warps = static_cast<long long>(rows) * ((H + Hkv + hpw - 1) / hpw);
+  if (warps > 0x7fffffffll) return -2;
   const dim3 grid(static_cast<unsigned>((warps + 7) / 8));
-#define RPEG_RA(T_, P_)                                                                                                               \
-  return launch_pdl(rotary_append_kernel<T_, P_>, grid, dim3(256), 0, STREAM(stream), src, splits, stride, ld, q_col0, k_col0, v_col0, slot, \
-                    pos, cos_t, sin_t, page_table, max_pages, static_cast<T_*>(q_out), ldq, static_cast<T_*>(kcache),                  \
+#define RPEG_RA(T_, P_, H_)                                                                                                           \
+  return launch_pdl(rotary_append_kernel<T_, P_, H_>, grid, dim3(256), 0, STREAM(stream), src, splits, stride, ld, q_col0, k_col0, v_col0, \
+                    slot, pos, cos_t, sin_t, page_table, max_pages, static_cast<T_*>(q_out), ldq, static_cast<T_*>(kcache),            \
                     static_cast<T_*>(vcache), rows, H, Hkv, dim, dp, rot_dims, do_norm, eps) == cudaSuccess ? 0 : -21;
-  if (f32) { RPEG_RA(float, false) }
-  if (splits > 0) { RPEG_RA(__nv_bfloat16, true) }
-  RPEG_RA(__nv_bfloat16, false)
+  if (f32) { RPEG_RA(float, false, 1) }
+  if (splits > 0) { RPEG_RA(__nv_bfloat16, true, 1) }
+  if (hpw == 4) { RPEG_RA(__nv_bfloat16, false, 4) }
+  RPEG_RA(__nv_bfloat16, false, 1)
 #undef RPEG_RA
 }
 

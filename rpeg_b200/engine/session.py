@@ -39,8 +39,6 @@ class Session:
     # ------------------------------------------------------------------ pages
     def _reserve(self, q: _Request, n: int) -> None:
         """Pages for ``n`` more tokens of the request."""
-        if q.length + n > self.gen.max_seq_len:
-            raise ValueError(f"a request of {q.length + n} tokens exceeds max_seq_len ({self.gen.max_seq_len})")
         have = q.gone + len(q.pages)
         need = -(-(q.length + n) // PAGE) - have
         if need > 0:
@@ -89,10 +87,14 @@ class Session:
                 raise ValueError(f"request {rid!r} brings a token outside the vocabulary")
             if len(want) and (min(want) < 0 or max(want) >= len(tokens)):
                 raise ValueError(f"request {rid!r} wants a place outside its tokens")
-            if rid not in self.requests:
-                if not self.free_slots:
-                    raise RuntimeError(f"all {g.max_slots} slots are taken")
-                self.requests[rid] = _Request(self.free_slots.pop())
+            have = self.requests[rid].length if rid in self.requests else 0
+            if have + len(tokens) > g.max_seq_len:
+                raise ValueError(f"request {rid!r} of {have + len(tokens)} tokens exceeds max_seq_len ({g.max_seq_len})")
+        new = [rid for rid, _, _ in entries if rid not in self.requests]
+        if len(new) > len(self.free_slots):
+            raise RuntimeError(f"{len(new)} new requests but only {len(self.free_slots)} of {g.max_slots} slots are free")
+        for rid in new:
+            self.requests[rid] = _Request(self.free_slots.pop())
         reqs = [self.requests[rid] for rid, _, _ in entries]
         for q, (_, tokens, _) in zip(reqs, entries):
             self._reserve(q, len(tokens))

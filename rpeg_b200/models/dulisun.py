@@ -310,10 +310,14 @@ class DulisunModel:
         return self._run(tokens, pos, slot, page_table, kcache, vcache, attend, False, trace)
 
     def _nsplit(self, m: AttentionMixer, rows: int, table_pages: int) -> int:
-        """Splits that give every SM about two CTAs, at most one per page a row can see."""
+        """Splits of a decode row's pages: the fewest page times over all waves of CTAs, where a CTA costs about four pages on
+        top of its own (pipeline fill, merge) and two or three of them share an SM."""
         pages = min(table_pages, m.window // K.KV_PAGE + 2) if m.window else table_pages
-        ctas = rows * m.kv_heads * -(-(m.heads // m.kv_heads) // 8)
-        return max(1, min(-(-2 * self._num_sms // ctas), pages, 32))
+        group = m.heads // m.kv_heads
+        narrow = (group - 1) % 8 < 4 and group <= 12
+        ctas = rows * m.kv_heads * -(-group // (4 if narrow else 8))
+        slots = self._num_sms * (3 if narrow else 2)
+        return min(range(1, min(pages, 16) + 1), key=lambda n: (-(-ctas * n // slots) * (-(-pages // n) + 4), n))
 
     def _split_buffers(self, rows: int, table_pages: int) -> Tuple[torch.Tensor, torch.Tensor]:
         """Scratch of the split attention for ``rows`` rows; kept for good, captured graphs point into it."""
