@@ -51,6 +51,9 @@ def load_hf_config(model_dir) -> Dict[str, Any]:
 
 
 def model_spec_from_hf_config(cfg: Dict[str, Any], parameter_count: Optional[int] = None) -> ModelSpec:
+    if "architecture" in cfg:
+        raise RuntimeConfigError(f"the planner's cost model covers decoders of equal dense layers, not {cfg['architecture']!r} models "
+                                 "(they are served through engine.generate and engine.session)")
     hidden, heads = int(cfg["hidden_size"]), int(cfg["num_attention_heads"])
     return ModelSpec(int(cfg["num_hidden_layers"]), hidden, int(cfg["intermediate_size"]), int(cfg["vocab_size"]), 2,
                      int(cfg.get("head_dim") or hidden // heads), parameter_count)

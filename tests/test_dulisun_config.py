@@ -28,6 +28,12 @@ def test_config_reads_every_size_and_round_trips():
     assert cfg.kv_geometry() == [(3, 24, 24), (1, 40, 40), (4, 136, 136), (2, 64, 64)]
 
 
+def test_planner_refuses_the_family_with_a_reason():
+    from rpeg_b200.runtime.hf import model_spec_from_hf_config
+    with pytest.raises(RuntimeConfigError, match="cost model"):
+        model_spec_from_hf_config(C.regular())
+
+
 @pytest.mark.parametrize("path,value,word", [
     (("layers", 0, "type"), "recurrent", "mixer type"), (("layers", 0, "mixer", "kv_heads"), 4, "divide"),
     (("layers", 0, "mixer", "vdim"), 24, "vdim"), (("layers", 0, "mixer", "dim"), 300, "dim"), (("layers", 0, "mixer", "rot", "dims"), 13, "rot"),
