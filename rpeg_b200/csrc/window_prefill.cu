@@ -6,25 +6,33 @@
 // (window = 0: [0, p]). The portion's own keys were appended to the cache before, so a whole prompt, a portion of one
 // and a batch of unequal portions are the same launch: nothing depends on where a prompt was cut.
 //
-// One CTA = 128 query rows of one head; the pipeline is the one of flash_attn.cu (TMA warp, MMA warp, four softmax
-// warps; S double buffered in TMEM, P in TMEM columns of its own, lazy rescaling of O). Differences:
-//   * a key tile is two 64-token cache pages, fetched by TMA through the request's page-table row; tiles start at the
-//     page that holds the first key any row of the CTA sees;
-//   * heads narrower than the tile (64 or 128) are padded by the TMA unit (out-of-bounds columns read as zero);
-//   * the sink opens the softmax: the running maximum starts no lower than the sink's logit and the running sum with its
+// One CTA works on two 128-row query tiles ("units") over the same key tiles: the same rows of two heads of one KV head,
+// or, when the KV head has an odd number of query heads, two neighbouring row tiles of one head. While the softmax warps of one
+// unit turn its scores into weights, the tensor cores multiply for the other one. Roles: a TMA warp, an MMA warp, four softmax
+// warps per unit (thread = query row).
+//   * TMEM: S (128 columns) and O (up to 128) of each unit. A unit's weights replace its scores in place, 32-key chunk by
+//     chunk: a weight is handed to the tensor cores as the sum of two bf16 numbers (16 bits), so that rounding the operands
+//     of P V does not show; its two parts take 16 of the chunk's 32 columns each.
+//   * The commit behind Q K^T of a unit's next tile also covers that unit's P V before it, so the softmax warps need no
+//     other signal before they rescale O or overwrite S.
+//   * O is rescaled only when a row's maximum grew by more than 8 (log2); a stale reference is exact after the final division.
+//   * A key tile is two 64-token cache pages, fetched by TMA through the request's page-table row; tiles start at the page that
+//     holds the first key any row of the CTA sees. Heads narrower than the tile (64 or 128) are padded by the TMA unit
+//     (out-of-bounds columns read as zero).
+//   * The sink opens the softmax: the running maximum starts no lower than the sink's logit and the running sum with its
 //     exponential, so it needs no key and no pass of its own.
-#include "common.cuh"
+#include "act_io.cuh"
 #include "rpeg_kernels.h"
 
 namespace rpeg {
 
-constexpr int WP_BM = 128, WP_BN = 128, WP_THREADS = 192, WP_STAGES = 2;
+constexpr int WP_BM = 128, WP_BN = 128, WP_THREADS = 320, WP_STAGES = 2;
 constexpr float WP_RESCALE = 8.0f;
 
 template <int HDT>
 struct PrefillCfg {
   static constexpr int TILE = 128 * HDT * 2;               // HDT / 64 atoms of 128 rows x 128 bytes
-  static constexpr int SMEM = TILE * (1 + 2 * WP_STAGES) + 1024 + 256;
+  static constexpr int SMEM = TILE * (2 + 2 * WP_STAGES) + 1024 + 256;
 };
 
 struct Prefill {
@@ -33,64 +41,81 @@ struct Prefill {
   const float* sink;
   __nv_bfloat16* out; int ldo;
   int H, Hkv, dp, window;
+  int pair_heads;                           // units: two heads of one KV head (1) or two row tiles of one head (0)
   float scale_log2;
   int* status;
 };
 
-// Largest raw score of the row among the visible keys [lo, hi] of the tile that starts at k0.
-template <bool MASK>
-__device__ __forceinline__ float wp_max_pass(uint32_t ts, int k0, int lo, int hi) {
-  uint32_t a[32], b[32];
-  float tmax = -INFINITY;
-  tmem_ld_32x32(ts, a);
+// A row's 128 scores of one tile, in registers from the maximum to the weights: S is read from TMEM once.
+struct WpRow {
+  uint32_t s[4][32];
+};
+
+__device__ __forceinline__ void wp_load_row(uint32_t ts, WpRow& row) {
 #pragma unroll
-  for (int c = 0; c < 4; ++c) {
-    tmem_wait_ld();
-    uint32_t(&cur)[32] = (c & 1) ? b : a;
-    if (c + 1 < 4) tmem_ld_32x32(ts + (c + 1) * 32, (c & 1) ? a : b);
+  for (int c = 0; c < 4; ++c) tmem_ld_32x32(ts + c * 32, row.s[c]);
+  tmem_wait_ld();
+}
+
+// Keys outside [lo, hi] of the tile that starts at k0 get no weight, whatever their (finite or not) score is.
+__device__ __forceinline__ void wp_mask_row(WpRow& row, int k0, int lo, int hi) {
+#pragma unroll
+  for (int c = 0; c < 4; ++c)
 #pragma unroll
     for (int i = 0; i < 32; ++i) {
       const int kj = k0 + c * 32 + i;
-      if (!MASK || (kj >= lo && kj <= hi)) tmax = fmaxf(tmax, __uint_as_float(cur[i]));
+      if (kj < lo || kj > hi) row.s[c][i] = 0xff800000u;
     }
-  }
-  return tmax;
 }
 
-// P = exp2(s * scale - m_ref) as packed bf16, its row sum, and the largest raw score seen.
-template <bool MASK>
-__device__ __forceinline__ void wp_exp_pass(uint32_t ts, uint32_t tp, float scale_log2, float m_ref, int k0, int lo, int hi, float& lsum,
-                                            float& smax) {
-  uint32_t a[32], b[32];
-  tmem_ld_32x32(ts, a);
+__device__ __forceinline__ float wp_max_row(const WpRow& row) {
+  float m[4];
 #pragma unroll
   for (int c = 0; c < 4; ++c) {
-    tmem_wait_ld();
-    uint32_t(&cur)[32] = (c & 1) ? b : a;
-    if (c + 1 < 4) tmem_ld_32x32(ts + (c + 1) * 32, (c & 1) ? a : b);
-    uint32_t pk[16];
+    m[c] = __uint_as_float(row.s[c][0]);
+#pragma unroll
+    for (int i = 1; i < 32; ++i) m[c] = fmaxf(m[c], __uint_as_float(row.s[c][i]));
+  }
+  return fmaxf(fmaxf(m[0], m[1]), fmaxf(m[2], m[3]));
+}
+
+// P = exp2(s * scale - m_ref) over S in place (columns 32 c .. + 15: leading parts of chunk c, + 16 .. + 31: remainders);
+// returns its row sum. `half_bar` gets this warp's arrival once the first 64 keys are in place.
+__device__ __forceinline__ float wp_exp_row(const WpRow& row, uint32_t ts, float scale_log2, float m_ref, uint64_t* half_bar) {
+  const uint64_t scale2 = pack2(scale_log2, scale_log2), shift2 = pack2(-m_ref, -m_ref), minus2 = pack2(-1.f, -1.f);
+  uint64_t sum2[2] = {0ull, 0ull};
+#pragma unroll
+  for (int c = 0; c < 4; ++c) {
+    uint32_t head[16], rest[16];
 #pragma unroll
     for (int i = 0; i < 16; ++i) {
-      const int kj = k0 + c * 32 + 2 * i;
-      const float s0 = __uint_as_float(cur[2 * i]), s1 = __uint_as_float(cur[2 * i + 1]);
-      float p0, p1;
-      if (MASK) {
-        const bool v0 = kj >= lo && kj <= hi, v1 = kj + 1 >= lo && kj + 1 <= hi;
-        if (v0) smax = fmaxf(smax, s0);
-        if (v1) smax = fmaxf(smax, s1);
-        p0 = v0 ? exp2f(fmaf(s0, scale_log2, -m_ref)) : 0.f;
-        p1 = v1 ? exp2f(fmaf(s1, scale_log2, -m_ref)) : 0.f;
-      } else {
-        smax = fmaxf(smax, fmaxf(s0, s1));
-        p0 = exp2f(fmaf(s0, scale_log2, -m_ref));
-        p1 = exp2f(fmaf(s1, scale_log2, -m_ref));
-      }
-      lsum += p0 + p1;
-      pk[i] = pack_bf16x2(p0, p1);
+      const float2 t = unpack2(fma2(pack2(__uint_as_float(row.s[c][2 * i]), __uint_as_float(row.s[c][2 * i + 1])), scale2, shift2));
+      const float p0 = exp2f(t.x), p1 = exp2f(t.y);
+      const uint64_t p = pack2(p0, p1);
+      sum2[i & 1] = add2(sum2[i & 1], p);
+      // leading part: the upper 16 bits as they are; the remainder is exact in fp32 and rounded to bf16
+      const uint32_t w0 = __float_as_uint(p0), w1 = __float_as_uint(p1);
+      head[i] = __byte_perm(w0, w1, 0x7632);
+      const float2 r = unpack2(fma2(pack2(__uint_as_float(w0 & 0xffff0000u), __uint_as_float(w1 & 0xffff0000u)), minus2, p));
+      rest[i] = pack_bf16x2(r.x, r.y);
     }
-    tmem_st_32x16(tp + c * 16, pk);
+    tmem_st_32x16(ts + c * 32, head);
+    tmem_st_32x16(ts + c * 32 + 16, rest);
+    if (c == 1) {
+      tmem_wait_st();
+      tc_fence_before_sync();
+      __syncwarp();
+      if ((threadIdx.x & 31) == 0) mbar_arrive(half_bar);
+    }
   }
+  const float2 s0 = unpack2(sum2[0]), s1 = unpack2(sum2[1]);
+  return (s0.x + s0.y) + (s1.x + s1.y);
 }
+
+// One unit: its rows' positions and the key tiles [jb, je) of the CTA that any of its rows sees (je = jb: absent).
+struct PrefillUnit {
+  int h, q0, p0, p_last, last_lo, jb, je;
+};
 
 template <int HDT>
 __global__ void __launch_bounds__(WP_THREADS, 1)
@@ -98,23 +123,34 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
                       const __grid_constant__ CUtensorMap tmap_v, const Prefill a) {
   using Cfg = PrefillCfg<HDT>;
   constexpr int ATOMS = HDT / 64, TILE = Cfg::TILE;
-  const int b = blockIdx.z, h = blockIdx.y;
-  const int qt = gridDim.x - 1 - blockIdx.x;
+  const int b = blockIdx.z;
+  const int bx = gridDim.x - 1 - blockIdx.x;                // late tiles have the most keys: first
   const int tok0 = a.cu[b], L = a.cu[b + 1] - tok0;
-  const int q0 = qt * WP_BM;
-  if (q0 >= L) return;
-  const int hk = h / (a.H / a.Hkv);
-  const int p0 = a.pos[tok0] + q0;                          // position of the CTA's first row
-  const int p_last = p0 + min(WP_BM, L - q0) - 1;
-  const int first_key = a.window > 0 ? p0 / a.window * a.window : 0;
-  const int last_lo = a.window > 0 ? p_last / a.window * a.window : 0;
-  const int kb = first_key & ~(RPEG_KV_PAGE - 1);
-  const int n_tiles = (p_last + 1 - kb + WP_BN - 1) / WP_BN;
+  const int q_first = bx * (a.pair_heads ? WP_BM : 2 * WP_BM);
+  if (q_first >= L) return;
+  const int start = a.pos[tok0];
+  const int kb = (a.window > 0 ? (start + q_first) / a.window * a.window : 0) & ~(RPEG_KV_PAGE - 1);
+  auto unit = [&](int u) -> PrefillUnit {
+    PrefillUnit w;
+    w.h = a.pair_heads ? blockIdx.y * 2 + u : blockIdx.y;
+    w.q0 = a.pair_heads ? q_first : q_first + u * WP_BM;
+    w.p0 = start + w.q0;
+    w.p_last = w.p0 + min(WP_BM, L - w.q0) - 1;
+    const int first = a.window > 0 ? w.p0 / a.window * a.window : 0;
+    w.last_lo = a.window > 0 ? w.p_last / a.window * a.window : 0;
+    w.jb = (first - kb) > 0 ? (first - kb) / WP_BN : 0;
+    w.je = w.q0 < L ? (w.p_last - kb) / WP_BN + 1 : w.jb;
+    return w;
+  };
+  const PrefillUnit u0 = unit(0), u1 = unit(1);
+  const bool has1 = u1.je > u1.jb;
+  const int n_tiles = has1 ? max(u0.je, u1.je) : u0.je;
+  const int hk = u0.h / (a.H / a.Hkv);
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  uint8_t* q_sm = smem;
-  uint8_t* k_sm = smem + TILE;
+  uint8_t* q_sm = smem;                                      // [2]
+  uint8_t* k_sm = smem + 2 * TILE;
   uint8_t* v_sm = k_sm + WP_STAGES * TILE;
   uint64_t* bars = reinterpret_cast<uint64_t*>(v_sm + WP_STAGES * TILE);
   uint64_t* q_full = bars;
@@ -122,10 +158,11 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
   uint64_t* k_empty = k_full + WP_STAGES;
   uint64_t* v_full = k_empty + WP_STAGES;
   uint64_t* v_empty = v_full + WP_STAGES;
-  uint64_t* s_full = v_empty + WP_STAGES;   // [2]
-  uint64_t* p_full = s_full + 2;            // [2]
-  uint64_t* pv_done = p_full + 2;           // [2]: PV_j completes pv_done[j & 1]
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(pv_done + 2);
+  uint64_t* s_full = v_empty + WP_STAGES;   // [2], per unit: S of its next tile is complete (and its P V before that)
+  uint64_t* p_half = s_full + 2;            // [2], per unit: its weights for the first 64 keys are in place
+  uint64_t* p_full = p_half + 2;            // [2], per unit: and for the others
+  uint64_t* o_full = p_full + 2;            // [2], per unit: O is final
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(o_full + 2);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -135,7 +172,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
       mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1);
       mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1);
     }
-    for (int s = 0; s < 2; ++s) { mbar_init(&s_full[s], 1); mbar_init(&p_full[s], 4); mbar_init(&pv_done[s], 1); }
+    for (int u = 0; u < 2; ++u) { mbar_init(&s_full[u], 1); mbar_init(&p_half[u], 4); mbar_init(&p_full[u], 4); mbar_init(&o_full[u], 1); }
     *abort_flag = 0;
     fence_mbar_init();
   }
@@ -147,26 +184,31 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
   __syncthreads();
   tc_fence_after_sync();
   const uint32_t tmem_base = *tmem_slot;
-  const uint32_t tmem_o = tmem_base + 256;
 
   if (warp == 0) {
     if (lane == 0) {
       const int* pt = a.page_table + static_cast<size_t>(a.slot[tok0]) * a.max_pages;
+      const int last_key = has1 ? max(u0.p_last, u1.p_last) : u0.p_last;
       auto load_tile = [&](const CUtensorMap* map, uint8_t* dst, uint64_t* bar, int j) {
         mbar_expect_tx(bar, TILE);
 #pragma unroll
         for (int hf = 0; hf < 2; ++hf) {
           const int pi = kb / RPEG_KV_PAGE + 2 * j + hf;
           // a page past the row's last one is never visible: any valid page will do
-          const int page = pi * RPEG_KV_PAGE <= p_last ? pt[pi] : 0;
+          const int page = pi * RPEG_KV_PAGE <= last_key ? pt[pi] : 0;
           const int y = (page * a.Hkv + hk) * RPEG_KV_PAGE;
 #pragma unroll
           for (int c = 0; c < ATOMS; ++c) tma_load_2d(dst + c * 16384 + hf * 8192, map, bar, c * 64, y);
         }
       };
-      mbar_expect_tx(q_full, TILE);
+      mbar_expect_tx(q_full, has1 ? 2 * TILE : TILE);
 #pragma unroll
-      for (int c = 0; c < ATOMS; ++c) tma_load_3d(q_sm + c * 16384, &tmap_q, q_full, c * 64, h, tok0 + q0);
+      for (int u = 0; u < 2; ++u)
+        if (u == 0 || has1) {
+#pragma unroll
+          for (int c = 0; c < ATOMS; ++c)
+            tma_load_3d(q_sm + u * TILE + c * 16384, &tmap_q, q_full, c * 64, u ? u1.h : u0.h, tok0 + (u ? u1.q0 : u0.q0));
+        }
       for (int j = 0; j < n_tiles; ++j) {
         const int st = j % WP_STAGES;
         const uint32_t ph = static_cast<uint32_t>(j / WP_STAGES) & 1u;
@@ -180,119 +222,122 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
     if (lane == 0) {
       constexpr uint32_t idesc_qk = make_idesc_bf16(128, 128, 0, 0);
       constexpr uint32_t idesc_pv = make_idesc_bf16(128, HDT, 0, 1);
-      const uint32_t q_addr = smem_u32(q_sm);
-      auto issue_qk = [&](int j) {
+      auto active = [&](int u, int j) -> bool { return u == 0 ? j >= u0.jb && j < u0.je : has1 && j >= u1.jb && j < u1.je; };
+      // Q K^T of unit u over tile j; the tile's K buffer is free again once the last unit has used it
+      auto issue_qk = [&](int u, int j) {
         const int st = j % WP_STAGES;
-        const uint32_t k_addr = smem_u32(k_sm + st * TILE);
-        const uint32_t ts = tmem_base + static_cast<uint32_t>((j & 1) * 128);
+        if (active(u, j)) {
+          const uint32_t q_addr = smem_u32(q_sm + u * TILE), k_addr = smem_u32(k_sm + st * TILE);
 #pragma unroll
-        for (int k = 0; k < HDT / 16; ++k) {
-          const uint32_t off = static_cast<uint32_t>((k >> 2) * 16384 + (k & 3) * 32);
-          umma_bf16_ss(ts, make_smem_desc_sw128(q_addr + off, 16, 1024), make_smem_desc_sw128(k_addr + off, 16, 1024), idesc_qk,
-                       k != 0 ? 1u : 0u);
+          for (int k = 0; k < HDT / 16; ++k) {
+            const uint32_t off = static_cast<uint32_t>((k >> 2) * 16384 + (k & 3) * 32);
+            umma_bf16_ss(tmem_base + u * 128, make_smem_desc_sw128(q_addr + off, 16, 1024), make_smem_desc_sw128(k_addr + off, 16, 1024),
+                         idesc_qk, k != 0 ? 1u : 0u);
+          }
+          umma_commit(&s_full[u]);
         }
-        umma_commit(&k_empty[st]);
-        umma_commit(&s_full[j & 1]);
+        if (u == 1) umma_commit(&k_empty[st]);
       };
       bool ok = mbar_wait(q_full, 0, abort_flag, a.status, 910);
       if (ok) ok = mbar_wait(&k_full[0], 0, abort_flag, a.status, 911);
       if (ok) {
         tc_fence_after_sync();
-        issue_qk(0);
-        for (int j = 0; j < n_tiles; ++j) {
-          const int st = j % WP_STAGES;
-          const uint32_t ph = static_cast<uint32_t>(j / WP_STAGES) & 1u;
-          if (j + 1 < n_tiles) {
-            const int st1 = (j + 1) % WP_STAGES;
-            const uint32_t ph1 = static_cast<uint32_t>((j + 1) / WP_STAGES) & 1u;
-            if (!mbar_wait(&k_full[st1], ph1, abort_flag, a.status, 912)) break;
-            tc_fence_after_sync();
-            issue_qk(j + 1);
-          }
-          if (!mbar_wait(&p_full[j & 1], static_cast<uint32_t>(j >> 1) & 1u, abort_flag, a.status, 913)) break;
-          if (!mbar_wait(&v_full[st], ph, abort_flag, a.status, 914)) break;
-          tc_fence_after_sync();
+        issue_qk(0, 0);
+        issue_qk(1, 0);
+        for (int j = 0; j < n_tiles && ok; ++j) {
+          const int st = j % WP_STAGES, st1 = (j + 1) % WP_STAGES;
+          if (!mbar_wait(&v_full[st], static_cast<uint32_t>(j / WP_STAGES) & 1u, abort_flag, a.status, 915)) break;
+          if (j + 1 < n_tiles &&
+              !mbar_wait(&k_full[st1], static_cast<uint32_t>((j + 1) / WP_STAGES) & 1u, abort_flag, a.status, 912)) break;
           const uint32_t v_addr = smem_u32(v_sm + st * TILE);
-          const uint32_t tp = tmem_base + 384u + static_cast<uint32_t>((j & 1) * 64);
 #pragma unroll
-          for (int k = 0; k < 8; ++k)
-            umma_bf16_ts(tmem_o, tp + k * 8, make_smem_desc_sw128(v_addr + k * 2048, 16384, 1024), idesc_pv, (j | k) != 0 ? 1u : 0u);
-          umma_commit(&v_empty[st]);
-          umma_commit(&pv_done[j & 1]);
+          for (int u = 0; u < 2; ++u) {
+            if (active(u, j)) {
+              const int n = j - (u ? u1.jb : u0.jb);         // tiles of this unit before this one
+              const uint32_t tp = tmem_base + u * 128, to = tmem_base + 256 + u * 128;
+#pragma unroll
+              for (int half = 0; half < 2 && ok; ++half) {   // the first keys are multiplied while the last ones are exponentiated
+                ok = mbar_wait(half ? &p_full[u] : &p_half[u], static_cast<uint32_t>(n) & 1u, abort_flag, a.status, 913 + half);
+                if (!ok) break;
+                tc_fence_after_sync();
+#pragma unroll
+                for (int part = 0; part < 2; ++part)
+#pragma unroll
+                  for (int k = half * 4; k < half * 4 + 4; ++k)   // 16 keys: 8 packed columns of P, 16 rows (2 KiB) of the V tile
+                    umma_bf16_ts(to, tp + (k >> 1) * 32 + part * 16 + (k & 1) * 8, make_smem_desc_sw128(v_addr + k * 2048, 16384, 1024), idesc_pv,
+                                 (n | half | part | (k & 3)) != 0 ? 1u : 0u);
+              }
+              if (!ok) break;
+              if (j + 1 == (u ? u1.je : u0.je)) umma_commit(&o_full[u]);
+            }
+            if (u == 1) umma_commit(&v_empty[st]);
+            tc_fence_after_sync();
+            if (j + 1 < n_tiles) issue_qk(u, j + 1);
+          }
         }
       }
     }
   } else {
+    const int ui = (warp - 2) >> 2;
+    const PrefillUnit w = ui ? u1 : u0;
     const int quad = warp & 3;
     const int r = quad * 32 + lane;
-    const bool row_valid = q0 + r < L;
-    const int qi = p0 + r;
+    const bool row_valid = w.q0 + r < L;
+    const int qi = w.p0 + r;
     // an absent row sees nothing
     const int lo = row_valid ? (a.window > 0 ? qi / a.window * a.window : 0) : 1;
     const int hi = row_valid ? qi : 0;
-    const uint32_t lane_base = static_cast<uint32_t>(quad * 32) << 16;
-    const float sink_l2 = a.sink != nullptr ? a.sink[h] * 1.4426950408889634f : -INFINITY;
+    const uint32_t ts = tmem_base + (static_cast<uint32_t>(quad * 32) << 16) + ui * 128;
+    const uint32_t to = ts + 256;
+    const float sink_l2 = a.sink != nullptr ? a.sink[w.h] * 1.4426950408889634f : -INFINITY;
     float m_ref = -INFINITY, l = 0.f;
     bool ok = true;
-    // why a parity wait on pv_done is enough: see flash_attn.cu
-    auto wait_pv = [&](int tile, int where) -> bool {
-      return __all_sync(0xffffffffu, mbar_wait(&pv_done[tile & 1], static_cast<uint32_t>(tile >> 1) & 1u, abort_flag, a.status, where));
-    };
-    for (int j = 0; j < n_tiles && ok; ++j) {
-      const uint32_t ts = tmem_base + lane_base + static_cast<uint32_t>((j & 1) * 128);
-      const uint32_t tp = tmem_base + lane_base + 384u + static_cast<uint32_t>((j & 1) * 64);
-      if (!__all_sync(0xffffffffu, mbar_wait(&s_full[j & 1], static_cast<uint32_t>(j >> 1) & 1u, abort_flag, a.status, 920))) { ok = false; break; }
+    for (int j = w.jb; j < w.je; ++j) {
+      const int n = j - w.jb;
+      if (!__all_sync(0xffffffffu, mbar_wait(&s_full[ui], static_cast<uint32_t>(n) & 1u, abort_flag, a.status, 920))) { ok = false; break; }
       tc_fence_after_sync();
       const int k0 = kb + j * WP_BN;
-      const bool need_mask = k0 + WP_BN - 1 > p0 || k0 < last_lo || p_last - p0 < WP_BM - 1;
-      if (j == 0) {
-        // scale > 0, so the largest score is the scaled largest product
-        const float t0 = need_mask ? wp_max_pass<true>(ts, k0, lo, hi) : wp_max_pass<false>(ts, k0, lo, hi);
-        m_ref = fmaxf(t0 * a.scale_log2, sink_l2);
+      const bool need_mask = k0 + WP_BN - 1 > w.p0 || k0 < w.last_lo || w.p_last - w.p0 < WP_BM - 1;
+      // scale > 0, so the largest score is the scaled largest product
+      WpRow row;
+      wp_load_row(ts, row);
+      if (need_mask) wp_mask_row(row, k0, lo, hi);
+      const float tmax = wp_max_row(row) * a.scale_log2;
+      if (n == 0) {
+        m_ref = fmaxf(tmax, sink_l2);
         if (sink_l2 != -INFINITY) l = exp2f(sink_l2 - m_ref);
-      }
-      float lsum = 0.f, smax = -INFINITY;
-      // a row that has seen no key and has no sink keeps an infinite reference: whatever this pass gives it is
-      // recomputed below as soon as the tile holds a key it sees
-      if (need_mask) wp_exp_pass<true>(ts, tp, a.scale_log2, m_ref, k0, lo, hi, lsum, smax);
-      else wp_exp_pass<false>(ts, tp, a.scale_log2, m_ref, k0, lo, hi, lsum, smax);
-      if (j > 0) {
-        const float tmax = smax * a.scale_log2;
-        const bool need = smax != -INFINITY && tmax > m_ref + WP_RESCALE;
+      } else {
+        const bool need = tmax > m_ref + WP_RESCALE;
         if (__any_sync(0xffffffffu, need)) {
-          if (!wait_pv(j - 1, 921)) { ok = false; break; }
-          tc_fence_after_sync();
           const float alpha = need ? exp2f(m_ref - tmax) : 1.f;
           if (need) { m_ref = tmax; l *= alpha; }
 #pragma unroll 1
           for (int c = 0; c < HDT / 32; ++c) {
             uint32_t v[32];
-            tmem_ld_32x32(tmem_o + lane_base + c * 32, v);
+            tmem_ld_32x32(to + c * 32, v);
             tmem_wait_ld();
 #pragma unroll
             for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * alpha);
-            tmem_st_32x32(tmem_o + lane_base + c * 32, v);
+            tmem_st_32x32(to + c * 32, v);
           }
-          lsum = 0.f;
-          float unused = -INFINITY;
-          if (need_mask) wp_exp_pass<true>(ts, tp, a.scale_log2, m_ref, k0, lo, hi, lsum, unused);
-          else wp_exp_pass<false>(ts, tp, a.scale_log2, m_ref, k0, lo, hi, lsum, unused);
         }
       }
-      l += lsum;
+      // a row that has seen no key yet and has no sink: every weight of this tile is masked to zero
+      const float m_use = m_ref == -INFINITY ? 0.f : m_ref;
+      l += wp_exp_row(row, ts, a.scale_log2, m_use, &p_half[ui]);
       tmem_wait_st();
       tc_fence_before_sync();
       __syncwarp();
-      if (lane == 0) mbar_arrive(&p_full[j & 1]);
+      if (lane == 0) mbar_arrive(&p_full[ui]);
     }
-    if (ok && wait_pv(n_tiles - 1, 922)) {
+    if (ok && w.je > w.jb && __all_sync(0xffffffffu, mbar_wait(&o_full[ui], 0, abort_flag, a.status, 922))) {
       tc_fence_after_sync();
       const float inv_l = l > 0.f ? 1.f / l : 0.f;
-      __nv_bfloat16* orow = a.out + static_cast<size_t>(tok0 + q0 + r) * a.ldo + h * a.dp;
+      __nv_bfloat16* orow = a.out + static_cast<size_t>(tok0 + w.q0 + r) * a.ldo + w.h * a.dp;
 #pragma unroll 1
       for (int c = 0; c < HDT / 32; ++c) {
         uint32_t v[32];
-        tmem_ld_32x32(tmem_o + lane_base + c * 32, v);
+        tmem_ld_32x32(to + c * 32, v);
         tmem_wait_ld();
         if (row_valid) {
 #pragma unroll
@@ -335,7 +380,8 @@ static int launch_window_prefill(const CUtensorMap& tq, const CUtensorMap& tk, c
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, PrefillCfg<HDT>::SMEM) != cudaSuccess) return -20;
     configured = true;
   }
-  const dim3 grid((max_len + WP_BM - 1) / WP_BM, a.H, B);
+  const int rows_per_cta = a.pair_heads ? WP_BM : 2 * WP_BM;
+  const dim3 grid((max_len + rows_per_cta - 1) / rows_per_cta, a.pair_heads ? a.H / 2 : a.H, B);
   kern<<<grid, WP_THREADS, PrefillCfg<HDT>::SMEM, stream>>>(tq, tk, tv, a);
   return cudaGetLastError() == cudaSuccess ? 0 : -21;
 }
@@ -364,7 +410,7 @@ extern "C" int rpeg_window_prefill(const void* q, int ldq, const void* kcache, c
   rc = make_tmap_bf16_2d(&tv, vcache, dp, cache_rows, dp, 64, RPEG_KV_PAGE);
   if (rc) return rc - 200;
   const Prefill a{cu, pos, slot, page_table, max_pages, sink, static_cast<__nv_bfloat16*>(out), ldo, H, Hkv, dp, window,
-                  scale * 1.4426950408889634f, status};
+                  (H / Hkv) % 2 == 0 ? 1 : 0, scale * 1.4426950408889634f, status};
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   return dp <= 64 ? launch_window_prefill<64>(tq, tk, tv, a, B, max_len, st) : launch_window_prefill<128>(tq, tk, tv, a, B, max_len, st);
 }

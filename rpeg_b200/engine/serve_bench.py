@@ -183,10 +183,15 @@ def prefill_kernels(tab: Table, d, ll, T: int) -> None:
     pairs = T * (T + 1) / 2
     tab.add(ph, "llama flash attention", [lambda i=i: K.flash_attn_fwd(qkv[i], 0, lc.q_width, lc.q_width + lc.kv_width, cu, T, H, G, hd) for i in R],
             2 * T * (lc.qkv_width + H * hd), 4.0 * pairs * H * hd)
-    for window in sorted({T, max(128, T // 4)}, reverse=True):
+    short = max(128, T // 4)
+    cu4 = torch.arange(0, T + 1, short, **i32)
+    tab.add(ph, f"llama flash attention, sequences of {short}", [lambda i=i: K.flash_attn_fwd(qkv[i], 0, lc.q_width, lc.q_width + lc.kv_width, cu4, short, H, G, hd) for i in R],
+            2 * T * (lc.qkv_width + H * hd), 4.0 * (T // short) * short * (short + 1) / 2 * H * hd)
+    for window in (T, short):
         vis = sum(min(T - c, window) * (min(T - c, window) + 1) / 2 for c in range(0, T, window))
         tab.add(ph, f"paged prefill attention, chunk {window}", [lambda i=i: K.window_prefill(q[i], kc[i], vc[i], table, cu, pos, slot, T, H, window=window,
-                scale=hd ** -0.5, sink=d.sink[0]) for i in R], 2 * T * (2 * H + 2 * G) * hd, 4.0 * vis * H * hd, like="llama flash attention")
+                scale=hd ** -0.5, sink=d.sink[0]) for i in R], 2 * T * (2 * H + 2 * G) * hd, 4.0 * vis * H * hd,
+                like="llama flash attention" if window == T else f"llama flash attention, sequences of {short}")
     f = lc.d_ff
     tab.add(ph, "llama gate/up gemm + swiglu", [lambda i=i: K.gemm_swiglu(xb[i], ll.p[f"l{i % n}.w_gate_up"]) for i in R], 2 * (T * w + 2 * f * w + T * f), 4.0 * T * w * f)
     act = [torch.randn(T, f, **bf) for _ in R]

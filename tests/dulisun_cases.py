@@ -97,3 +97,15 @@ def worst_row(a, b):
     """Largest error of a row relative to the typical row norm: one wrong row among many shows."""
     a, b = a.double().cpu(), b.double().cpu()
     return ((a - b).norm(dim=-1).max() / b.norm(dim=-1).mean()).item()
+
+
+def worst_relative_row(a, b):
+    """Largest error of a row relative to its own norm (rows of very different size, e.g. averages over 1 to n values)."""
+    a, b = a.double().cpu(), b.double().cpu()
+    return ((a - b).norm(dim=-1) / (b.norm(dim=-1) + 1e-30)).max().item()
+
+
+def row_errors(a, b):
+    """Error of every row relative to the typical row norm."""
+    a, b = a.double().cpu(), b.double().cpu()
+    return (a - b).norm(dim=-1) / b.norm(dim=-1).mean()

@@ -89,26 +89,10 @@ def route(scores, router):
     return sorted(allowed, key=lambda e: -scores[e])[: router["top"]]
 
 
-def closeness(scores, router):
-    """How clear one token's choice is: the smallest ratio, in log units, between what was taken and the best of what was
-    left (over the groups and over the experts). A 16-bit run may decide a closer call differently."""
-    n, groups = router["experts"], router.get("groups") or {"count": 1, "keep": 1}
-    per, gap = n // groups["count"], math.inf
-    best = [max(scores[g * per:(g + 1) * per]) for g in range(groups["count"])]
-    order = sorted(best, reverse=True)
-    if groups["keep"] < len(order):
-        gap = math.log(order[groups["keep"] - 1] / order[groups["keep"]])
-    kept = sorted(range(groups["count"]), key=lambda g: -best[g])[: groups["keep"]]
-    free = sorted((scores[e] for e in range(n) if e // per in kept), reverse=True)
-    return min(gap, math.log(free[router["top"] - 1] / free[router["top"]])) if router["top"] < len(free) else gap
-
-
-def moe(h, t, pre, m, clear=None):
+def moe(h, t, pre, m):
     out = torch.zeros_like(h)
     s = torch.softmax(h @ t[pre + "router"].T, -1)
     for i in range(h.shape[0]):
-        if clear is not None:
-            clear[i] = min(clear[i], closeness(s[i].tolist(), m["router"]))
         for e in route(s[i].tolist(), m["router"]):
             out[i] += s[i, e] * ffn(h[i:i + 1], t, f"{pre}e{e}.")[0]
     if m.get("shared"):
@@ -116,18 +100,15 @@ def moe(h, t, pre, m, clear=None):
     return out
 
 
-def forward(config, tensors, tokens, layers_out=None, clear=None):
-    """Logits [tokens, vocab]; ``layers_out`` (a list) receives the residual stream after every layer, ``clear`` (a list)
-    the ``closeness`` of every token's closest routing decision."""
-    if clear is not None:
-        clear[:] = [math.inf] * len(tokens)
+def forward(config, tensors, tokens, layers_out=None):
+    """Logits [tokens, vocab]; ``layers_out`` (a list) receives the residual stream after every layer."""
     t = {k: v.to(F64) for k, v in tensors.items()}
     eps = config["norm"]["eps"]
     x = norm(t["embed"][torch.as_tensor(tokens, dtype=torch.long)], t["embed.norm"], eps)
     for i, layer in enumerate(config["layers"]):
         x = x + norm(attention(x, t, f"l{i}.mix.", layer["mixer"], eps), t[f"l{i}.norm1"], eps)
         if layer["mlp"] is not None:
-            x = x + norm(moe(x, t, f"l{i}.mlp.", layer["mlp"], clear), t[f"l{i}.norm2"], eps)
+            x = x + norm(moe(x, t, f"l{i}.mlp.", layer["mlp"]), t[f"l{i}.norm2"], eps)
         if layers_out is not None:
             layers_out.append(x)
     return norm(x, t["final.norm"], eps) @ t["embed"].T

@@ -23,6 +23,7 @@ from rpeg_b200.ops import kernels as K  # noqa: E402
 
 DT = (torch.float32, torch.bfloat16)
 TOL = {torch.float32: 2e-5, torch.bfloat16: 3e-2}
+ATTN = {torch.float32: 2e-5, torch.bfloat16: 5e-3}        # scores, weights and sums are fp32: only the output is rounded
 ROOT = Path(__file__).resolve().parent.parent
 
 
@@ -152,7 +153,7 @@ def _want(q, k, v, pos, window, scale, sink):
 
 @pytest.mark.parametrize("kernel", ["rows f32", "rows bf16", "rows bf16 split", "prefill"])
 @pytest.mark.parametrize("H,G,dim,window,sink", [(8, 2, 64, 0, True), (6, 1, 96, 120, True), (12, 1, 128, 200, False), (4, 4, 40, 64, True),
-                                                 (3, 3, 24, 7, True), (20, 2, 80, 129, True), (2, 1, 200, 90, True), (2, 2, 256, 0, False)])
+                                                 (3, 3, 24, 7, True), (20, 2, 80, 129, True), (9, 3, 48, 130, False), (2, 1, 200, 90, True), (2, 2, 256, 0, False)])
 def test_chunked_attention_with_sink(cuda_device, kernel, H, G, dim, window, sink):
     """Portions that start anywhere, two requests of unequal length, every row against the oracle."""
     if kernel == "prefill" and dim > K.WINDOW_PREFILL_MAX_DIM:
@@ -185,8 +186,31 @@ def test_chunked_attention_with_sink(cuda_device, kernel, H, G, dim, window, sin
         lens_t = (pos + 1).to(dev)
         lens_t[1] = 0
         o2 = K.rows_attn(q, kc, vc, table, slot, pos.to(dev), H, window=window, scale=scale, sink=skd, lens=lens_t)
-        assert o2[1].abs().sum() == 0 and C.worst_row(o2[2:], want[2:]) < TOL[dtype]
-    assert C.worst_row(out, want) < TOL[dtype]
+        assert o2[1].abs().sum() == 0 and C.worst_relative_row(o2[2:], want[2:]) < ATTN[dtype]
+    assert C.worst_relative_row(out, want) < ATTN[dtype]
+
+
+@pytest.mark.parametrize("H,G", [(3, 3), (4, 1), (3, 1)])
+@pytest.mark.parametrize("window,growing", [(0, False), (500, False), (512, True), (0, True)])
+def test_long_prompt_portions(cuda_device, H, G, window, growing):
+    """Many key tiles per row, two and more query tiles per portion; with ``growing`` the scores rise along the sequence, so
+    the running maximum (and the accumulator) is rescaled again and again."""
+    dev, dim, n, start, scale = cuda_device, 64, 1400, 333, 0.25
+    g = torch.Generator().manual_seed(H + window)
+    k, v = torch.randn(n, G, dim, generator=g), torch.randn(n, G, dim, generator=g)
+    q = torch.randn(n - start, H, dim, generator=g)
+    if growing:
+        k[..., 0] = torch.linspace(0.0, 40.0, n)[:, None]
+        q[..., 0] = 4.0
+    k, v, q = k.bfloat16(), v.bfloat16(), q.bfloat16()
+    kc, vc, table = _cache([k.float()], [v.float()], torch.bfloat16, dev)
+    pos = torch.arange(start, n, dtype=torch.int32)
+    sink = torch.randn(H, generator=g) if window else None
+    want = _want(q, k, v, pos, window, scale, sink)
+    out = K.window_prefill(q.reshape(len(pos), -1).to(dev), kc, vc, table, torch.tensor([0, n - start], dtype=torch.int32, device=dev), pos.to(dev),
+                           torch.zeros(n - start, dtype=torch.int32, device=dev), n - start, H, window=window, scale=scale,
+                           sink=None if sink is None else sink.to(dev))
+    assert C.worst_relative_row(out, want) < ATTN[torch.bfloat16]
 
 
 @pytest.mark.parametrize("kernel", ["rows", "prefill"])
@@ -217,7 +241,7 @@ def test_single_keys_at_chunk_and_page_edges(cuda_device, kernel, window):
         else:                                             # every row a portion of its own
             cu = torch.arange(len(ends) + 1, dtype=torch.int32, device=dev)
             got = K.window_prefill(qd, kc, vc, table, cu, pos.to(dev), slot, 1, H, window=window, scale=scale)
-        assert C.worst_row(got, want) < 2e-2, (spot, ends)
+        assert C.worst_relative_row(got, want) < ATTN[torch.bfloat16], (spot, ends)
         seen = torch.tensor([p // window == spot // window for p in ends])
         near = (got.float().cpu().view(len(ends), H, dim) - v[spot].bfloat16().float()).norm(dim=-1).mean(-1)
         assert (near[seen] < 0.1).all() and (near[~seen] > 1.0).all()
@@ -238,7 +262,7 @@ def test_sink_counts_once_in_the_denominator(cuda_device):
     for got in (K.window_prefill(q, kc, vc, table, cu, pos, slot, 130, 2, scale=0.7, sink=sink),
                 K.rows_attn(q, kc, vc, table, slot, pos, 2, scale=0.7, sink=sink),
                 K.rows_attn(q, kc, vc, table, slot, pos, 2, scale=0.7, sink=sink, nsplit=2, scratch=scratch, arrive=arrive)):
-        assert (got.float().cpu().view(130, 2, dim) - want[..., None]).abs().max() < 6e-3
+        assert (got.float().cpu().view(130, 2, dim) - want[..., None]).abs().max() < 2.5e-3
 
 
 # --------------------------------------------------------------------------- mixture of experts
@@ -339,29 +363,35 @@ def _feed(s, rid, tokens, sizes):
     return torch.cat(out)
 
 
+def _close(got, want, dtype):
+    """fp32: every row. bf16: rounding turns over the closest routing decisions (and the keys of such a token reach the next
+    few), so all but a few rows, and those few stay bounded."""
+    e = C.row_errors(got, want)
+    if dtype == torch.float32:
+        assert e.max() < 5e-5
+    else:
+        assert e.quantile(0.5) < 2e-2 and e.quantile(0.93) < 8e-2 and e.max() < 1.5
+
+
 @pytest.mark.parametrize("name,n", [("unlike", 260), ("regular", 200), ("long", 420)])
 def test_prefill_decode_and_portions_match_the_oracle(models, name, n):
     cfg, t, _, ms = models(name)
     tokens = _tokens(cfg, n, 1)
-    layers, clear = [], []
-    want = O.forward(cfg, t, tokens, layers, clear)
-    settled = torch.tensor(clear) > 0.05                   # rows whose routing no bf16 rounding turns over
-    assert settled.float().mean() > 0.5
+    layers = []
+    want = O.forward(cfg, t, tokens, layers)
     for dtype, model in ms.items():
-        rows = settled if dtype == torch.bfloat16 else torch.ones(n, dtype=torch.bool)
-        tol = {torch.float32: 5e-5, torch.bfloat16: 8e-2}[dtype]
         trace = []
         dev_tok = torch.tensor(tokens, dtype=torch.int32, device="cuda")
         xf, _ = model.forward(dev_tok, torch.arange(n, dtype=torch.int32, device="cuda"), torch.tensor([0, n], dtype=torch.int32, device="cuda"), n,
                               trace=trace)
-        assert max(C.rel(a[rows.cuda()], b[rows]) for a, b in zip(trace, layers)) < tol / 2
-        assert C.worst_row(model.lm_logits(xf).cpu()[rows], want[rows]) < tol
+        for a, b in zip(trace, layers):
+            _close(a, b, dtype)
+        _close(model.lm_logits(xf), want, dtype)
         s = _session(model)
         for sizes in ([n], [1], [n - 40, 1], [64], [2], [3, 61, 65, 2, 1, 1, 30, 7]):
             if dtype == torch.bfloat16 and sizes == [2]:
                 sizes = [2] * 20 + [n]
-            got = _feed(s, "r", tokens, sizes)
-            assert C.worst_row(got.cpu()[rows], want[rows]) < tol, (dtype, sizes)
+            _close(_feed(s, "r", tokens, sizes), want, dtype)
             s.end("r")                                    # the next pass runs on used pages
         assert s.gen.pool.available() == s.gen.pool.num_pages - 1
 
@@ -535,9 +565,5 @@ def test_replay_command(models, tmp_path, dtype):
     assert run.returncode == 0, run.stderr[-2000:]
     assert [ln for ln in run.stdout.splitlines() if ln.startswith("done ")] == [f"done {i}" for i in range(len(steps))]
     read = lambda i: torch.from_numpy(np.fromfile(tmp_path / f"{i}.f32", dtype="<f4")).view(-1, cfg["vocab"])  # noqa: E731
-    clear, cb = [], []
-    want = torch.cat([O.forward(cfg, t, a, clear=clear)[[0, 49, 50, 99] + list(range(102, 140))], O.forward(cfg, t, b, clear=cb)[[19]]])
-    got = torch.cat([read(0)] + [read(2 + i) for i in range(38)] + [read(1)])
-    gaps = torch.tensor([clear[i] for i in [0, 49, 50, 99] + list(range(102, 140))] + [cb[19]])
-    rows = gaps > (0.0 if dtype == "float32" else 0.05)
-    assert rows.sum() > 20 and C.worst_row(got[rows], want[rows]) < (5e-5 if dtype == "float32" else 8e-2)
+    want = torch.cat([O.forward(cfg, t, a)[[0, 49, 50, 99] + list(range(102, 140))], O.forward(cfg, t, b)[[19]]])
+    _close(torch.cat([read(0)] + [read(2 + i) for i in range(38)] + [read(1)]), want, getattr(torch, dtype))
