@@ -152,7 +152,7 @@ def _want(q, k, v, pos, window, scale, sink):
 
 
 @pytest.mark.parametrize("kernel", ["rows f32", "rows bf16", "rows bf16 split", "prefill"])
-@pytest.mark.parametrize("H,G,dim,window,sink", [(8, 2, 64, 0, True), (6, 1, 96, 120, True), (12, 1, 128, 200, False), (4, 4, 40, 64, True),
+@pytest.mark.parametrize("H,G,dim,window,sink", [(8, 2, 64, 0, True), (10, 2, 88, 112, True), (12, 1, 128, 200, False), (4, 4, 40, 64, True),
                                                  (3, 3, 24, 7, True), (20, 2, 80, 129, True), (9, 3, 48, 130, False), (2, 1, 200, 90, True), (2, 2, 256, 0, False)])
 def test_chunked_attention_with_sink(cuda_device, kernel, H, G, dim, window, sink):
     """Portions that start anywhere, two requests of unequal length, every row against the oracle."""
