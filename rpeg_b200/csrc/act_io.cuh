@@ -52,5 +52,25 @@ __device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
 
 // Exact (erf) gelu.
 __device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
+__device__ __forceinline__ float sigmoidf(float z) { return 1.f / (1.f + __expf(-z)); }
+// tanh to a few units in the last place (the compiler's fast-math tanhf is a 2^-11 approximation): Lambert's continued fraction
+// z / (1 + z^2 / (3 + z^2 / (5 + z^2 / (7 + z^2 / 9)))) near zero, 1 - 2 / (e^2z + 1) where nothing cancels.
+__device__ __forceinline__ float tanh_f32(float z) {
+  const float a = fabsf(z), q = z * z;
+  if (a < 0.55f) return z * (945.f + q * (105.f + q)) / (945.f + q * (420.f + 15.f * q));
+  return copysignf(1.f - 2.f / (1.f + __expf(2.f * a)), z);
+}
+
+// What a feed-forward's first product is followed by. Gated: the product has twice the columns (gate rows of the weight, then up
+// rows) and the result is silu(gate) * up.
+enum { FF_NONE = 0, FF_GELU = 1, FF_SWIGLU = 2, FF_RELU2 = 3 };
+
+template <int ACT>
+__device__ __forceinline__ float ff_act(float z) {
+  if constexpr (ACT == FF_GELU) return gelu_erf(z);
+  if constexpr (ACT == FF_RELU2) { const float r = fmaxf(z, 0.f); return r * r; }
+  return z;
+}
+__device__ __forceinline__ float silu_mul(float gate, float up) { return gate * sigmoidf(gate) * up; }
 
 }  // namespace rpeg

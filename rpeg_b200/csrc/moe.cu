@@ -1,13 +1,16 @@
 // Mixture of experts: routing, dispatch and the experts' matrix products.
 //
-//   moe_route      one warp per token: softmax over the router logits (fp32, from a GEMM output or its split-K
+//   moe_route      one warp per token: softmax or sigmoid of the router logits (fp32, from a GEMM output or its split-K
 //                  partials), the best groups of neighbouring experts by their largest score, the `top` largest scores
 //                  inside those groups; each choice takes a ticket of its expert's counter
-//   moe_dispatch   segment offsets from the counters, one copy of every chosen token's row into its expert's segment
+//   moe_dispatch   segment offsets from the counters, one copy of every chosen token's row into its expert's segment,
+//                  multiplied by the choice's weight if the weights belong to the experts' inputs
 //   moe_gemm       grouped GEMM on tcgen05: one persistent launch over the tiles of every expert's segment, the
 //                  number of rows of a segment is read on the device (nothing about the routing reaches the host, so a
-//                  decode step with a mixture is captured in a CUDA graph like any other); gelu in the epilogue
-// The weighted sum of a token's expert outputs is taken by the norm that follows (residual_norm.cu).
+//                  decode step with a mixture is captured in a CUDA graph like any other); gelu, squared relu or
+//                  silu(gate) * up in the epilogue. With one always-on segment it is a dense feed-forward's first product.
+// The (weighted) sum of a token's expert outputs is taken by the kernel that updates the residual stream (residual_norm.cu,
+// stream_update.cu).
 //
 // Equal scores: the expert (or group) with the smaller number wins.
 #include "act_io.cuh"
@@ -35,7 +38,7 @@ __device__ __forceinline__ int warp_argmax(const float* v, int n, uint32_t mask,
 
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const float* __restrict__ logits, int splits, long long stride, int ld, int rows, int E, int n_groups, int keep, int top,
-                 int renorm, int* __restrict__ ids, float* __restrict__ wts, int* __restrict__ ticket, int* __restrict__ counts) {
+                 int renorm, int sigmoid, int* __restrict__ ids, float* __restrict__ wts, int* __restrict__ ticket, int* __restrict__ counts) {
   griddep_launch();
   griddep_wait();
   extern __shared__ float route_sm[];
@@ -54,15 +57,19 @@ moe_route_kernel(const float* __restrict__ logits, int splits, long long stride,
     sc[e] = z;
     mx = fmaxf(mx, z);
   }
-  mx = warp_max(mx);
-  float sum = 0.f;
-  for (int e = lane; e < E; e += 32) {
-    const float p = expf(sc[e] - mx);
-    sc[e] = p;
-    sum += p;
+  if (sigmoid) {
+    for (int e = lane; e < E; e += 32) sc[e] = sigmoidf(sc[e]);
+  } else {
+    mx = warp_max(mx);
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) {
+      const float p = expf(sc[e] - mx);
+      sc[e] = p;
+      sum += p;
+    }
+    const float inv = 1.f / warp_sum(sum);
+    for (int e = lane; e < E; e += 32) sc[e] *= inv;
   }
-  const float inv = 1.f / warp_sum(sum);
-  for (int e = lane; e < E; e += 32) sc[e] *= inv;
   __syncwarp();
   const int per = E / n_groups;
   uint32_t open = 0xffffffffu;                             // bit j: expert lane + 32 j may still be chosen (E <= 1024)
@@ -101,9 +108,22 @@ moe_route_kernel(const float* __restrict__ logits, int splits, long long stride,
 }
 
 // One CTA per token. Every CTA sums the counters below its token's experts itself (a few hundred words from L2).
+// `wts`: weights of the choices, multiplied into the copies (null: plain copies).
+__device__ __forceinline__ uint4 scaled(uint4 v, float w, const float*) {
+  return make_uint4(__float_as_uint(__uint_as_float(v.x) * w), __float_as_uint(__uint_as_float(v.y) * w), __float_as_uint(__uint_as_float(v.z) * w),
+                    __float_as_uint(__uint_as_float(v.w) * w));
+}
+__device__ __forceinline__ uint4 scaled(uint4 v, float w, const __nv_bfloat16*) {
+  auto two = [&](uint32_t u) -> uint32_t {
+    const float2 f = unpack_bf16x2(u);
+    return pack_bf16x2(f.x * w, f.y * w);
+  };
+  return make_uint4(two(v.x), two(v.y), two(v.z), two(v.w));
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128)
-moe_dispatch_kernel(const T* __restrict__ x, int dp, const int* __restrict__ ids, const int* __restrict__ ticket,
+moe_dispatch_kernel(const T* __restrict__ x, int dp, const int* __restrict__ ids, const int* __restrict__ ticket, const float* __restrict__ wts,
                     const int* __restrict__ counts, int E, int top, T* __restrict__ xs, int* __restrict__ row_of, int* __restrict__ seg_off) {
   griddep_launch();
   griddep_wait();
@@ -140,12 +160,15 @@ moe_dispatch_kernel(const T* __restrict__ x, int dp, const int* __restrict__ ids
   const uint4* src = reinterpret_cast<const uint4*>(x + static_cast<size_t>(t) * dp);
   for (int i = threadIdx.x; i < nv; i += blockDim.x) {
     const uint4 v = src[i];
-    for (int k = 0; k < top; ++k) reinterpret_cast<uint4*>(xs + static_cast<size_t>(rows_sm[k]) * dp)[i] = v;
+    for (int k = 0; k < top; ++k)
+      reinterpret_cast<uint4*>(xs + static_cast<size_t>(rows_sm[k]) * dp)[i] = wts == nullptr ? v : scaled(v, wts[static_cast<size_t>(t) * top + k], x);
   }
 }
 
 // ---------------------------------------------------------------------------------- grouped GEMM
 //   C[r, 0..N) = act( A[r, 0..K) * B_s[0..N, 0..K)^T )   for every row r of segment s;  B_s = rows [s * N, s * N + N) of B
+// (gated: B_s has 2 N rows, gate then up; a tile of BN accumulator columns holds BN / 2 gate columns and the BN / 2 up columns of
+// the same outputs)
 // Same structure as the dense kernel in gemm.cu (TMA producer warp, one MMA-issuing thread, four epilogue warps,
 // accumulator double buffered in TMEM). A tile is 128 rows of ONE segment: it starts at any row (the row coordinate
 // of a TMA box is free) and the rows that belong to the next segment are computed and not stored. Always-on
@@ -163,13 +186,14 @@ struct MoeGemmCfg {
   static constexpr int SMEM_BYTES = STAGES * STAGE_BYTES + 1024 + 512 + (MOE_MAX_SEGMENTS + 1) * 4;
 };
 
-template <int BN, bool GELU>
+template <int BN, int ACT>
 __global__ void __launch_bounds__(MG_THREADS, 1)
 moe_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ CUtensorMap tmap_x,
                 const __grid_constant__ CUtensorMap tmap_b, __nv_bfloat16* __restrict__ C, const int* __restrict__ seg_off, int n_routed,
                 int n_shared, int seg_rows, int shared_from_x, int N, int K, int ldc, int a_rows, int* status) {
   using Cfg = MoeGemmCfg<BN>;
   constexpr int STAGES = Cfg::STAGES;
+  constexpr int TN = ACT == FF_SWIGLU ? BN / 2 : BN;   // output columns per tile
   const uint32_t stage_tx = static_cast<uint32_t>(Cfg::B_BYTES + a_rows * MG_BK * 2);
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -220,7 +244,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constan
   __syncthreads();
   tc_fence_after_sync();
   const uint32_t tmem_base = *tmem_slot;
-  const int n_tiles = (N + BN - 1) / BN;
+  const int n_tiles = (N + TN - 1) / TN;
   const int num_items = mt0[S] * n_tiles;
   const int num_kb = (K + MG_BK - 1) / MG_BK;
 
@@ -247,12 +271,14 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constan
         const bool from_x = shared_from_x && it.seg >= n_routed;
         const CUtensorMap* ta = from_x ? &tmap_x : &tmap_a;
         const int m0 = it.tm * MG_BM + (from_x ? 0 : static_cast<int>(sg.row0));
-        const int b0 = it.seg * N + it.tn * BN;
+        const int b0 = it.seg * (ACT == FF_SWIGLU ? 2 * N : N) + it.tn * TN;
         for (int kb = 0; kb < num_kb; ++kb) {
           if (!mbar_wait(&empty_bar[stage], phase ^ 1u, abort_flag, status, 700)) goto producer_done;
           uint8_t* sa = smem + stage * Cfg::STAGE_BYTES;
           mbar_expect_tx(&full_bar[stage], stage_tx);
           tma_load_2d(sa + Cfg::A_BYTES, &tmap_b, &full_bar[stage], kb * MG_BK, b0);
+          if constexpr (ACT == FF_SWIGLU)      // the boxes are TN rows high: gate rows, then the up rows of the same columns
+            tma_load_2d(sa + Cfg::A_BYTES + TN * MG_BK * 2, &tmap_b, &full_bar[stage], kb * MG_BK, b0 + N);
           tma_load_2d(sa, ta, &full_bar[stage], kb * MG_BK, m0);
           if (++stage == STAGES) { stage = 0; phase ^= 1u; }
         }
@@ -295,18 +321,19 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constan
       const int r = it.tm * MG_BM + quad * 32 + lane;
       const bool live = r < sg.rows;
       const bool warp_live = it.tm * MG_BM + quad * 32 < sg.rows;    // decode: most quads of a tile hold no row at all
-      const int n0 = it.tn * BN;
+      const int n0 = it.tn * TN;
       if (!__all_sync(0xffffffffu, mbar_wait(&tfull_bar[buf], acc_phase, abort_flag, status, 720))) break;
       tc_fence_after_sync();
       const uint32_t taddr = tmem_base + (static_cast<uint32_t>(quad * 32) << 16) + static_cast<uint32_t>(buf * BN);
       if (warp_live) {
         __nv_bfloat16* crow = C + static_cast<size_t>(sg.row0 + r) * ldc;
 #pragma unroll 1
-        for (int c = 0; c < BN / 32; ++c) {
+        for (int c = 0; c < TN / 32; ++c) {
           const int col0 = n0 + c * 32;
           if (col0 >= N) break;                                      // uniform over the warp
-          uint32_t v[32];
+          uint32_t v[32], u[ACT == FF_SWIGLU ? 32 : 1];
           tmem_ld_32x32(taddr + c * 32, v);
+          if constexpr (ACT == FF_SWIGLU) tmem_ld_32x32(taddr + TN + c * 32, u);
           tmem_wait_ld();
           if (live) {
 #pragma unroll
@@ -316,7 +343,13 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constan
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                   float a = __uint_as_float(v[q * 8 + 2 * e]), b = __uint_as_float(v[q * 8 + 2 * e + 1]);
-                  if (GELU) { a = gelu_erf(a); b = gelu_erf(b); }
+                  if constexpr (ACT == FF_SWIGLU) {
+                    a = silu_mul(a, __uint_as_float(u[q * 8 + 2 * e]));
+                    b = silu_mul(b, __uint_as_float(u[q * 8 + 2 * e + 1]));
+                  } else {
+                    a = ff_act<ACT>(a);
+                    b = ff_act<ACT>(b);
+                  }
                   o[e] = pack_bf16x2(a, b);
                 }
                 *reinterpret_cast<uint4*>(crow + col0 + q * 8) = make_uint4(o[0], o[1], o[2], o[3]);
@@ -345,12 +378,12 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constan
 int make_tmap_bf16_2d(CUtensorMap* out, const void* ptr, uint64_t inner, uint64_t outer, uint64_t ld, uint32_t box_inner,
                       uint32_t box_outer);
 
-template <int BN, bool GELU>
+template <int BN, int ACT>
 static int launch_moe_gemm(const CUtensorMap& ta, const CUtensorMap& tx, const CUtensorMap& tb, void* C, const int* seg_off, int n_routed,
                            int n_shared, int seg_rows, int from_x, int N, int K, int ldc, int a_rows, long long max_tiles, int num_sms,
                            int* status, cudaStream_t stream) {
   using Cfg = MoeGemmCfg<BN>;
-  auto kern = moe_gemm_kernel<BN, GELU>;
+  auto kern = moe_gemm_kernel<BN, ACT>;
   static bool configured = false;
   if (!configured) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES) != cudaSuccess) return -20;
@@ -368,34 +401,34 @@ using namespace rpeg;
 #define STREAM(s) reinterpret_cast<cudaStream_t>(s)
 
 extern "C" int rpeg_moe_route(const float* logits, int splits, long long stride, int ld, int rows, int E, int n_groups, int keep, int top,
-                              int renorm, int* ids, float* wts, int* ticket, int* counts, void* stream) {
+                              int renorm, int sigmoid, int* ids, float* wts, int* ticket, int* counts, void* stream) {
   if (rows <= 0) return 0;
   if (E < 1 || n_groups < 1 || E % n_groups || keep < 1 || keep > n_groups || top < 1 || top > keep * (E / n_groups)) return -2;
   if (E > MOE_MAX_SEGMENTS) return -3;
   const size_t smem = static_cast<size_t>(ROUTE_WARPS) * (E + n_groups + top) * 4;
   if (smem > 48 * 1024) return -3;
   const cudaError_t e = launch_pdl(moe_route_kernel, dim3((rows + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem,
-                                   STREAM(stream), logits, splits, stride, ld, rows, E, n_groups, keep, top, renorm, ids, wts, ticket, counts);
+                                   STREAM(stream), logits, splits, stride, ld, rows, E, n_groups, keep, top, renorm, sigmoid, ids, wts, ticket, counts);
   return e == cudaSuccess ? 0 : -21;
 }
 
-extern "C" int rpeg_moe_dispatch(const void* x, int dp, const int* ids, const int* ticket, const int* counts, int rows, int E, int top,
-                                 void* xs, int* row_of, int* seg_off, int f32, void* stream) {
+extern "C" int rpeg_moe_dispatch(const void* x, int dp, const int* ids, const int* ticket, const float* wts, const int* counts, int rows,
+                                 int E, int top, void* xs, int* row_of, int* seg_off, int f32, void* stream) {
   if (rows <= 0) return 0;
   if ((dp & 7) || E < 1 || E > MOE_MAX_SEGMENTS || top < 1 || top > E) return -2;
   const size_t smem = static_cast<size_t>(E + 1 + top) * 4;
   const cudaError_t e =
       f32 ? launch_pdl(moe_dispatch_kernel<float>, dim3(rows), dim3(128), smem, STREAM(stream), static_cast<const float*>(x), dp, ids, ticket,
-                       counts, E, top, static_cast<float*>(xs), row_of, seg_off)
+                       wts, counts, E, top, static_cast<float*>(xs), row_of, seg_off)
           : launch_pdl(moe_dispatch_kernel<__nv_bfloat16>, dim3(rows), dim3(128), smem, STREAM(stream), static_cast<const __nv_bfloat16*>(x),
-                       dp, ids, ticket, counts, E, top, static_cast<__nv_bfloat16*>(xs), row_of, seg_off);
+                       dp, ids, ticket, wts, counts, E, top, static_cast<__nv_bfloat16*>(xs), row_of, seg_off);
   return e == cudaSuccess ? 0 : -21;
 }
 
 // A [a_rows_total, K]: routed rows (and the always-on ones unless X is given); X [seg_rows, K] or null; B [(n_routed +
-// n_shared) * N, K]; C rows as A's segments. `choices` = routed rows in total (seg_rows * top), for the grid size.
+// n_shared) * N, K] (2 N rows per segment for FF_SWIGLU); C rows as A's segments. `choices` = routed rows in total (seg_rows * top), for the grid size.
 extern "C" int rpeg_moe_gemm(const void* A, long long a_rows_total, const void* X, const void* B, void* C, const int* seg_off, int n_routed,
-                             int n_shared, int seg_rows, long long choices, int N, int K, int lda, int ldx, int ldb, int ldc, int gelu,
+                             int n_shared, int seg_rows, long long choices, int N, int K, int lda, int ldx, int ldb, int ldc, int act,
                              int bn_hint, int* status, void* stream) {
   if (seg_rows <= 0 || N <= 0 || K <= 0) return 0;
   const int S = n_routed + n_shared;
@@ -417,23 +450,31 @@ extern "C" int rpeg_moe_gemm(const void* A, long long a_rows_total, const void* 
   if (bn == 0) {
     // widest tile that still gives every SM one, unless it wastes much more of the last column tile than a narrower one
     bn = 256;
-    while (bn > 64 && (m_tiles * ((N + bn - 1) / bn) < num_sms || (N + bn - 1) / bn * bn * 8 > ((N + 127) / 128 * 128) * 9)) bn >>= 1;
+    const int cols = act == FF_SWIGLU ? 2 * N : N;
+    while (bn > 64 && (m_tiles * ((cols + bn - 1) / bn) < num_sms || (cols + bn - 1) / bn * bn * 8 > ((cols + 127) / 128 * 128) * 9)) bn >>= 1;
   }
+  const int tn = act == FF_SWIGLU ? bn / 2 : bn;
   const int a_rows = seg_rows <= 32 ? 32 : (seg_rows <= 64 ? 64 : MG_BM);
   CUtensorMap ta, tx, tb;
   int rc = make_tmap_bf16_2d(&ta, A, K, a_rows_total, lda, MG_BK, a_rows);
   if (rc) return rc;
   rc = X != nullptr ? make_tmap_bf16_2d(&tx, X, K, seg_rows, ldx, MG_BK, a_rows) : make_tmap_bf16_2d(&tx, A, K, a_rows_total, lda, MG_BK, a_rows);
   if (rc) return rc - 100;
-  rc = make_tmap_bf16_2d(&tb, B, K, static_cast<uint64_t>(S) * N, ldb, MG_BK, bn);
+  rc = make_tmap_bf16_2d(&tb, B, K, static_cast<uint64_t>(S) * N * (act == FF_SWIGLU ? 2 : 1), ldb, MG_BK, tn);
   if (rc) return rc - 200;
-  const long long max_tiles = m_tiles * ((N + bn - 1) / bn);
-#define RPEG_MG_CASE(BN_)                                                                                                          \
-  case BN_:                                                                                                                        \
-    return gelu ? launch_moe_gemm<BN_, true>(ta, tx, tb, C, seg_off, n_routed, n_shared, seg_rows, X != nullptr, N, K, ldc, a_rows, \
-                                             max_tiles, num_sms, status, STREAM(stream))                                           \
-                : launch_moe_gemm<BN_, false>(ta, tx, tb, C, seg_off, n_routed, n_shared, seg_rows, X != nullptr, N, K, ldc,       \
-                                              a_rows, max_tiles, num_sms, status, STREAM(stream));
+  const long long max_tiles = m_tiles * ((N + tn - 1) / tn);
+#define RPEG_MG_ACT(BN_, ACT_)                                                                                                       \
+  return launch_moe_gemm<BN_, ACT_>(ta, tx, tb, C, seg_off, n_routed, n_shared, seg_rows, X != nullptr, N, K, ldc, a_rows, max_tiles, \
+                                    num_sms, status, STREAM(stream));
+#define RPEG_MG_CASE(BN_)                             \
+  case BN_:                                           \
+    switch (act) {                                    \
+      case FF_NONE: RPEG_MG_ACT(BN_, FF_NONE)         \
+      case FF_GELU: RPEG_MG_ACT(BN_, FF_GELU)         \
+      case FF_SWIGLU: RPEG_MG_ACT(BN_, FF_SWIGLU)     \
+      case FF_RELU2: RPEG_MG_ACT(BN_, FF_RELU2)       \
+      default: return -4;                             \
+    }
   switch (bn) {
     RPEG_MG_CASE(256)
     RPEG_MG_CASE(128)
@@ -441,5 +482,6 @@ extern "C" int rpeg_moe_gemm(const void* A, long long a_rows_total, const void* 
     default:
       return -4;
   }
+#undef RPEG_MG_ACT
 #undef RPEG_MG_CASE
 }

@@ -14,50 +14,10 @@
 // Weights are stored either as they are applied or as the difference from one (`w_add` is 0 or 1).
 // One CTA per row, the row in registers between the passes. Rows are padded to a multiple of 8 columns
 // (`dp`); the padding holds zeros and stays zero, the mean is over the true width `d`.
-#include "act_io.cuh"
+#include "stream_source.cuh"
 #include "rpeg_kernels.h"
 
 namespace rpeg {
-
-enum { NSRC_ACT = 0, NSRC_PARTIALS = 1, NSRC_MOE = 2, NSRC_EMBED = 3, NSRC_STREAM = 4 };
-
-struct NormSource {
-  const void* p;            // activation / partials / expert rows / table / stream
-  int splits;               // partials: how many, `stride` floats apart
-  long long stride;
-  int ld;                   // row pitch in elements
-  const int* idx;           // token ids, or the expert-output row of every (token, choice)
-  const float* wts;         // weight of every (token, choice)
-  int top, n_shared;        // choices per token; always-on experts: rows shared_row0 + s * rows + t, weight 1
-  long long shared_row0;
-};
-
-template <typename T, int SRC>
-__device__ __forceinline__ float4 norm_source(const NormSource& s, const int* choice_row, const float* choice_w, int row, int rows, int c) {
-  if constexpr (SRC == NSRC_PARTIALS) {
-    const float* p = static_cast<const float*>(s.p) + static_cast<size_t>(row) * s.ld + c;
-    float4 v = load4(p);
-#pragma unroll 8
-    for (int k = 1; k < s.splits; ++k) v = add4(v, load4(p + k * s.stride));
-    return v;
-  } else if constexpr (SRC == NSRC_MOE) {
-    const T* y = static_cast<const T*>(s.p) + c;
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 8
-    for (int k = 0; k < s.top + s.n_shared; ++k) {
-      const float w = choice_w[k];
-      const float4 e = load4(y + static_cast<size_t>(choice_row[k]) * s.ld);
-      v.x = fmaf(w, e.x, v.x); v.y = fmaf(w, e.y, v.y); v.z = fmaf(w, e.z, v.z); v.w = fmaf(w, e.w, v.w);
-    }
-    return v;
-  } else if constexpr (SRC == NSRC_EMBED) {
-    return load4(static_cast<const T*>(s.p) + static_cast<size_t>(s.idx[row]) * s.ld + c);
-  } else if constexpr (SRC == NSRC_STREAM) {
-    return load4(static_cast<const float*>(s.p) + static_cast<size_t>(row) * s.ld + c);
-  } else {
-    return load4(static_cast<const T*>(s.p) + static_cast<size_t>(row) * s.ld + c);
-  }
-}
 
 __device__ __forceinline__ float block_sum(float v, float* part) {
   v = warp_sum(v);
@@ -99,7 +59,7 @@ residual_norm_kernel(const NormSource src, const T* __restrict__ w, const T* __r
       const bool routed = k < src.top;
       choice_row[k] = routed ? src.idx[static_cast<size_t>(row) * src.top + k]
                              : static_cast<int>(src.shared_row0 + static_cast<long long>(k - src.top) * rows + row);
-      choice_w[k] = routed ? src.wts[static_cast<size_t>(row) * src.top + k] : 1.f;
+      choice_w[k] = routed && src.wts != nullptr ? src.wts[static_cast<size_t>(row) * src.top + k] : 1.f;
     }
     __syncthreads();
   }

@@ -189,17 +189,51 @@ int rpeg_window_prefill(const void* q, int ldq, const void* kcache, const void* 
 
 // ---- moe.cu: mixture of experts (routing, dispatch, grouped GEMM over the experts' row segments)
 int rpeg_moe_route(const float* logits, int splits, long long stride, int ld, int rows, int E, int n_groups, int keep, int top,
-                   int renorm, int* ids, float* wts, int* ticket, int* counts, void* stream);
-int rpeg_moe_dispatch(const void* x, int dp, const int* ids, const int* ticket, const int* counts, int rows, int E, int top,
-                      void* xs, int* row_of, int* seg_off, int f32, void* stream);
+                   int renorm, int sigmoid, int* ids, float* wts, int* ticket, int* counts, void* stream);
+int rpeg_moe_dispatch(const void* x, int dp, const int* ids, const int* ticket, const float* wts, const int* counts, int rows, int E,
+                      int top, void* xs, int* row_of, int* seg_off, int f32, void* stream);
 int rpeg_moe_gemm(const void* A, long long a_rows_total, const void* X, const void* B, void* C, const int* seg_off, int n_routed,
-                  int n_shared, int seg_rows, long long choices, int N, int K, int lda, int ldx, int ldb, int ldc, int gelu,
+                  int n_shared, int seg_rows, long long choices, int N, int K, int lda, int ldx, int ldb, int ldc, int act,
                   int bn_hint, int* status, void* stream);
 
 // ---- gemm_f32.cu: fp32 matrix products on the CUDA cores
 int rpeg_gemm_f32(const float* A, const float* B, float* C, int M, int N, int K, int lda, int ldb, int ldc, void* stream);
 int rpeg_moe_gemm_f32(const float* A, const float* X, const float* B, float* C, const int* seg_off, int n_routed, int n_shared,
-                      int seg_rows, int N, int K, int lda, int ldb, int ldc, int gelu, void* stream);
+                      int seg_rows, int N, int K, int lda, int ldb, int ldc, int act, void* stream);
+int rpeg_gemm_f32_batched(const float* A, const float* B, float* C, int M, int N, int K, int lda, int ldb, int ldc, long long a_stride,
+                          long long b_stride, long long c_stride, int batch, int b_kn, void* stream);
+
+// ---- stream_update.cu: x += mixer output + feed-forward output; y = tanh(alpha x) w + b (fp32 stream, see the source for the kinds)
+int rpeg_stream_update(int kind_a, const void* a, int splits_a, long long stride_a, int ld_a, const int* ids, int kind_b, const void* b,
+                       int splits_b, long long stride_b, int ld_b, const int* row_of, const float* wts, int top, int n_shared,
+                       long long shared_row0, const float* alpha, const void* w, const void* bias, float* x, void* y, int rows, int dp,
+                       int f32, void* stream);
+
+// ---- latent.cu: latent attention around the projections, and on the CUDA cores
+int rpeg_latent_rows(const void* src, int splits, long long stride, int ld, int rows, const int* pos, const int* slot, const float* cos_t,
+                     const float* sin_t, int rot, int rot_p, float eps, int nq_col0, int nq, int nq_p, const void* nq_w, void* nq_out,
+                     int kv_col0, int rank, int rank_p, const void* kv_w, void* cache, const int* page_table, int max_pages, int q_col0,
+                     int H, int dim_p, void* q_nope, int ld_nope, void* q_rot, int ld_rot, int hs_rot, int f32, void* stream);
+int rpeg_latent_gather(const void* cache, int row_bytes, const int* page_table, int max_pages, const int* slot, const int* cu, const int* off,
+                       const int* lo, int B, int rows, void* out, void* stream);
+int rpeg_latent_attn_rows(const void* q, const void* cache, const int* page_table, int max_pages, const int* slot, const int* pos,
+                          const int* lens, const float* sink, void* out, int rows, int H, int rank_p, int W, int window, float scale, int f32,
+                          void* stream);
+
+// ---- latent_decode.cu / latent_prefill.cu: the same on the tensor cores
+int rpeg_latent_decode_ctas(int rank_p, int W);
+long long rpeg_latent_decode_scratch(int rows, int H, int rank_p, int nsplit);
+int rpeg_latent_decode(const void* q, const void* cache, long long num_pages, const int* page_table, int max_pages, const int* slot, const int* pos,
+                       const int* lens, const float* sink, void* out, float* scratch, int rows, int H, int rank_p, int W, int window, int nsplit,
+                       float scale, int* status, void* stream);
+int rpeg_latent_prefill_fits(int dim_p, int rot_p, int vdim_p);
+int rpeg_latent_prefill(const void* q, int ldq, int hsq, const void* kv, const void* rows, long long n_rows, int W, int rank_p, const int* cu,
+                        const int* pos, const int* off, const int* lo, const float* sink, void* out, int ldo, int T, int B, int max_len, int H,
+                        int dim_p, int rot_p, int vdim_p, int window, float scale, int* status, void* stream);
+
+// ---- head_gemm.cu: C[r, h, :] = A[r, h, :] * B_h
+int rpeg_head_gemm(const void* A, const void* B, void* C, int M, int N, int K, int H, int lda, int hsa, int ldc, int hsc, int b_kn, int* status,
+                   void* stream);
 
 #ifdef __cplusplus
 }

@@ -16,7 +16,7 @@ Design (B200-first):
 Models name their cache layout (``kv_geometry``: heads and widths per layer) and may offer two things more:
   * ``cached_prefill``: prompts attend over the paged cache, so they can be fed in portions (``prefill_portion`` bounds
     the tokens of a row one forward takes; ``engine.session`` feeds arbitrary ones);
-  * ``first_visible_key(pos)``: keys below it are never read again (chunked attention). Pages that lie below it are given
+  * ``first_visible_key(pos)``: keys below it are never read again (chunked or sliding attention). Pages that lie below it are given
     back to the pool while the row still runs.
 Semantics kept from the reference's quantile-phase generation (:2370-2628): rows end at EOS or at
 the length cap; outputs are returned per original row index, right padded, with a response mask.
@@ -235,7 +235,8 @@ class Generator:
         seq_id = torch.cat([torch.full((l,), s, dtype=torch.int32) for l, s in zip(lens, slots)]).to(dev)
         cu = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32, device=dev)
         if self.cached_prefill:
-            return self.model.prefill(tokens, pos, cu, max(lens), seq_id, self.page_table, self.kcache, self.vcache), cu
+            kw = {"spans": (starts, lens)} if getattr(self.model, "prefill_spans", False) else {}
+            return self.model.prefill(tokens, pos, cu, max(lens), seq_id, self.page_table, self.kcache, self.vcache, **kw), cu
         if any(starts):
             raise ValueError("this model prefills whole prompts only")
 
@@ -339,7 +340,7 @@ class Generator:
         self.row_key0.zero_()
         slot_row = [-1] * n
         slot_pages: List[List[int]] = [[] for _ in range(n)]   # pages a slot owns (the shared prompt pages are not in here)
-        slot_gone = [0] * n        # pages behind the shared ones that the row has passed for good (chunked attention)
+        slot_gone = [0] * n        # pages behind the shared ones that the row has passed for good (chunked or sliding attention)
         slot_shared = [0] * n      # leading page-table entries that alias the group's shared prompt pages
         slot_bound = [0] * n       # upper bound on the tokens a slot holds (prompt + decode steps run since admission)
         slot_prompt = [0] * n

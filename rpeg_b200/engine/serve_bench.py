@@ -210,9 +210,9 @@ def prefill_kernels(tab: Table, d, ll, T: int) -> None:
         rt.append((ids, wts, tk, c, K.moe_dispatch(xb[i], ids, wts, tk, c, e.experts)))
     tab.add(ph, "dispatch", [lambda i=i: K.moe_dispatch(xb[i], *rt[i][:4], e.experts) for i in R], 2 * T * w * (1 + e.top), like="llama rmsnorm + residual")
     rows, seg = T * (e.top + e.n_shared), e.segments
-    tab.add(ph, "experts up gemm + gelu", [lambda i=i: K.moe_gemm(rt[i][4].x_sorted, d.p[f"l{i % n}.w_up"], rt[i][4], e.experts, e.n_shared, shared_x=xb[i], gelu=True) for i in R],
+    tab.add(ph, "experts up gemm + gelu", [lambda i=i: K.moe_gemm(rt[i][4].x_sorted, d.p[f"l{i % n}.w_up"], rt[i][4], e.experts, e.n_shared, shared_x=xb[i], act="gelu") for i in R],
             2 * (T * w * (1 + e.top) + seg * e.ff * w + rows * e.ff), 2.0 * rows * w * e.ff, like="llama gate/up gemm + swiglu")
-    up = [K.moe_gemm(rt[i][4].x_sorted, d.p[f"l{i % n}.w_up"], rt[i][4], e.experts, e.n_shared, shared_x=xb[i], gelu=True) for i in R]
+    up = [K.moe_gemm(rt[i][4].x_sorted, d.p[f"l{i % n}.w_up"], rt[i][4], e.experts, e.n_shared, shared_x=xb[i], act="gelu") for i in R]
     tab.add(ph, "experts down gemm", [lambda i=i: K.moe_gemm(up[i], d.p[f"l{i % n}.w_down"], rt[i][4], e.experts, e.n_shared) for i in R],
             2 * (rows * e.ff + seg * e.ff * w + rows * w), 2.0 * rows * w * e.ff, like="llama down gemm")
     ys = [K.MoEOutput(K.moe_gemm(up[i], d.p[f"l{i % n}.w_down"], rt[i][4], e.experts, e.n_shared), rt[i][4].row_of, rt[i][4].weights, e.n_shared) for i in R]
@@ -283,9 +283,9 @@ def decode_kernels(tab: Table, d, ll, B: int, ctx: int) -> None:
     tab.add(ph, "route", [lambda: K.moe_route(lg, e.experts, e.top, c0, n_groups=e.groups, keep_groups=e.keep) for _ in L], 4.0 * B * (e.experts + 3 * e.top), like="llama swiglu")
     tab.add(ph, "dispatch", [lambda i=i: K.moe_dispatch(h, *rt[i][:4], e.experts) for i in L], 2.0 * B * w * (1 + e.top), like="llama rmsnorm + residual")
     used = sum(int((r[3] > 0).sum()) for r in rt) / n + e.n_shared
-    tab.add(ph, "experts up gemm + gelu", [lambda i=i: K.moe_gemm(rt[i][4].x_sorted, d.p[f"l{i}.w_up"], rt[i][4], e.experts, e.n_shared, shared_x=h, gelu=True) for i in L],
+    tab.add(ph, "experts up gemm + gelu", [lambda i=i: K.moe_gemm(rt[i][4].x_sorted, d.p[f"l{i}.w_up"], rt[i][4], e.experts, e.n_shared, shared_x=h, act="gelu") for i in L],
             used * wbytes(e.ff, w), like="llama gate/up gemm (split-K)")
-    up = [K.moe_gemm(rt[i][4].x_sorted, d.p[f"l{i}.w_up"], rt[i][4], e.experts, e.n_shared, shared_x=h, gelu=True) for i in R]
+    up = [K.moe_gemm(rt[i][4].x_sorted, d.p[f"l{i}.w_up"], rt[i][4], e.experts, e.n_shared, shared_x=h, act="gelu") for i in R]
     tab.add(ph, "experts down gemm", [lambda i=i: K.moe_gemm(up[i], d.p[f"l{i}.w_down"], rt[i][4], e.experts, e.n_shared) for i in L], used * wbytes(e.ff, w),
             like="llama down gemm (split-K)")
     ys = [K.MoEOutput(K.moe_gemm(up[i], d.p[f"l{i}.w_down"], rt[i][4], e.experts, e.n_shared), rt[i][4].row_of, rt[i][4].weights, e.n_shared) for i in R]

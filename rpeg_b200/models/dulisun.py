@@ -18,23 +18,19 @@ What runs where:
   * a shared feed-forward wider than the routed experts is stored as several always-on experts of their size (its hidden
     units are independent), so routed and shared experts are one grouped GEMM up and one down.
 
-Matrix rows and columns are padded to multiples of 8 elements with zeros (16-byte rows for TMA), so any size loads.
 This family is served (generation, log-probs); it has no backward pass here.
 """
 from __future__ import annotations
 
 import math
 from dataclasses import dataclass
-from typing import Dict, List, Optional, Tuple
+from typing import Dict, Iterable, List, Optional, Tuple
 
 import torch
 
 from ..ops import kernels as K
 from .llama import FlatLayout
-
-
-def pad8(n: int) -> int:
-    return (n + 7) // 8 * 8
+from .served import ServedDecoder, pad8
 
 
 @dataclass(frozen=True)
@@ -145,34 +141,18 @@ class DulisunLayout(FlatLayout):
         self.add("final_norm", d)
 
 
-class DulisunModel:
-    """Weights and kernels of one model on one GPU, with the interface the generator drives."""
+class DulisunModel(ServedDecoder):
+    """Weights and kernels of one model on one GPU."""
 
-    cached_prefill = True               # prompts may be fed in portions: attention reads the paged cache
-    needs_finite_cache = True           # tensor-core tiles cover whole pages: stale entries must be finite numbers
     KERNEL_SOURCES = ("gemm.cu", "generate.cu", "loss.cu", "residual_norm.cu", "window_attn.cu", "window_prefill.cu", "moe.cu", "gemm_f32.cu")
 
     def __init__(self, cfg: DulisunConfig, device, *, dtype: torch.dtype = torch.bfloat16, seed: Optional[int] = 0,
                  trainable: bool = False):
         """``seed=None`` leaves the weights zero (a checkpoint is about to be loaded)."""
-        if trainable:
-            raise ValueError("the dulisun family has no backward pass: it is served, not trained")
-        if dtype not in (torch.bfloat16, torch.float32):
-            raise ValueError(f"dtype {dtype} is not supported (bfloat16 or float32)")
-        self.cfg, self.device, self.dtype = cfg, torch.device(device), dtype
-        self.f32 = dtype == torch.float32
-        self.layout = DulisunLayout(cfg)
-        self.w = torch.zeros(self.layout.total, dtype=dtype, device=self.device)
-        self.p: Dict[str, torch.Tensor] = {n: self.layout.view(self.w, n) for n in self.layout.entries}
+        super().__init__(cfg, DulisunLayout(cfg), device, dtype=dtype, trainable=trainable)
         self.sink = [torch.zeros(l.mixer.heads, dtype=torch.float32, device=self.device) for l in cfg.layers]
         self.max_experts = max([l.mlp.experts for l in cfg.layers if l.mlp is not None], default=1)
-        self._ws: Optional[torch.Tensor] = None
         self._split: Dict[Tuple[int, int], Tuple[torch.Tensor, torch.Tensor]] = {}
-        self._tables: Dict[Tuple[float, int], Tuple[torch.Tensor, torch.Tensor]] = {}
-        self._outgrown: List[dict] = []      # tables that captured graphs may still read
-        self.positions = 0
-        self.reserve_positions(cfg.max_pos)
-        self._num_sms = torch.cuda.get_device_properties(self.device).multi_processor_count if self.device.type == "cuda" else 148
         if seed is not None:
             self.init_weights(seed)
 
@@ -226,45 +206,23 @@ class DulisunModel:
             self.put_expert(i, e.experts + s, up[s * e.ff:(s + 1) * e.ff], down[:, s * e.ff:(s + 1) * e.ff])
 
     # ------------------------------------------------------------------ what the generator asks
-    def kv_geometry(self) -> List[Tuple[int, int, int]]:
-        return self.cfg.kv_geometry()
+    def rotations(self) -> Iterable[Tuple[float, int]]:
+        return [(l.mixer.rot_base, l.mixer.rot_dims) for l in self.cfg.layers]
 
-    def reserve_positions(self, n: int) -> None:
-        """Make the rotary tables cover positions below ``n`` (a generator reserves its longest row when it is built)."""
-        if n <= self.positions:
-            return
-        self.positions = n
-        self._outgrown.append(self._tables)
-        self._tables = {}
-        for l in self.cfg.layers:
-            key = (l.mixer.rot_base, l.mixer.rot_dims)
-            if l.mixer.rot_dims:
-                self._tables[key] = K.rope_tables(n, l.mixer.rot_dims, l.mixer.rot_base, self.device)
+    def head_weight(self) -> torch.Tensor:
+        return self.p["embed"]
 
     def first_visible_key(self, pos: int) -> int:
         """Smallest position any layer still reads once every later token stands at ``pos`` or beyond."""
         return min((pos // l.mixer.window * l.mixer.window if l.mixer.window else 0) for l in self.cfg.layers)
 
     # ------------------------------------------------------------------ forward
-    def _workspace(self) -> torch.Tensor:
-        if self._ws is None:
-            self._ws = torch.empty(32 * 1024 * 1024, dtype=torch.float32, device=self.device)
-        return self._ws
-
-    def _lin(self, x: torch.Tensor, w: torch.Tensor, decode: bool, f32_out: bool = False):
-        """A projection: split-K partials for few rows (the consumer sums them), a plain GEMM otherwise."""
-        if self.f32:
-            return K.gemm_f32(x, w)
-        if decode:
-            return K.gemm_partials(x, w, self._workspace())
-        return K.gemm(x, w, out_dtype=torch.float32 if f32_out else torch.bfloat16)
-
     def _mixture(self, i: int, e: ExpertMixture, h: torch.Tensor, counts: torch.Tensor, decode: bool) -> K.MoEOutput:
         p = self.p
         logits = self._lin(h, p[f"l{i}.router"], decode, f32_out=True)
         ids, wts, ticket = K.moe_route(logits, e.experts, e.top, counts, n_groups=e.groups, keep_groups=e.keep)
         r = K.moe_dispatch(h, ids, wts, ticket, counts, e.experts)
-        act = K.moe_gemm(r.x_sorted, p[f"l{i}.w_up"], r, e.experts, e.n_shared, shared_x=h if e.n_shared else None, gelu=True)
+        act = K.moe_gemm(r.x_sorted, p[f"l{i}.w_up"], r, e.experts, e.n_shared, shared_x=h if e.n_shared else None, act="gelu")
         y = K.moe_gemm(act, p[f"l{i}.w_down"], r, e.experts, e.n_shared)
         return K.MoEOutput(y, r.row_of, r.weights, e.n_shared)
 
@@ -340,38 +298,3 @@ class DulisunModel:
                                sink=self.sink[i], nsplit=self._nsplit(m, B, table_pages), scratch=scratch, arrive=arrive)
 
         return self._run(token, pos, slot_ids, page_table, kcache, vcache, attend, True)
-
-    def forward(self, tokens, pos, cu_seqlens, max_seqlen: int, keep: bool = False, kv_sink=None, h_in=None, trace=None):
-        """Packed whole sequences without a generator's cache: the keys go to scratch pages that every layer reuses.
-        ``trace`` (a list) receives the residual stream after every layer."""
-        if keep or kv_sink is not None or h_in is not None:
-            raise ValueError("the dulisun family runs whole sequences for inference only")
-        lens = [int(v) for v in (cu_seqlens[1:] - cu_seqlens[:-1]).tolist()]
-        self.reserve_positions(max(lens))
-        pages = [-(-l // K.KV_PAGE) for l in lens]
-        table = torch.zeros((len(lens), max(pages)), dtype=torch.int32)
-        first = 1
-        for b, n in enumerate(pages):
-            table[b, :n] = torch.arange(first, first + n, dtype=torch.int32)
-            first += n
-        slot = torch.repeat_interleave(torch.arange(len(lens), dtype=torch.int32), torch.tensor(lens)).to(self.device)
-        geom = self.kv_geometry()
-        store = torch.zeros((2, max(first * h * K.KV_PAGE * max(dk, dv) for h, dk, dv in geom)), dtype=self.dtype, device=self.device)
-        kc = [store[0, : first * h * K.KV_PAGE * dk].view(first, h, K.KV_PAGE, dk) for h, dk, _ in geom]
-        vc = [store[1, : first * h * K.KV_PAGE * dv].view(first, h, K.KV_PAGE, dv) for h, _, dv in geom]
-        return self.prefill(tokens, pos, cu_seqlens, max(lens), slot, table.to(self.device), kc, vc, trace), None
-
-    # ------------------------------------------------------------------ heads
-    def lm_logits(self, xf: torch.Tensor, decode: bool = False) -> torch.Tensor:
-        """Logits ``[rows, vocab]`` against the embedding table (bf16, or fp32 in an fp32 model)."""
-        if self.f32:
-            return K.gemm_f32(xf, self.p["embed"])[:, : self.cfg.vocab]
-        return K.gemm(xf, self.p["embed"], workspace=self._workspace() if decode else None)[:, : self.cfg.vocab]
-
-    def token_logprobs(self, xf_rows: torch.Tensor, targets: torch.Tensor, chunk: int = 8192, temperature: float = 1.0) -> torch.Tensor:
-        """``log p(target)`` of the given hidden rows, at most ``chunk`` rows of logits at a time."""
-        out = torch.empty(xf_rows.shape[0], dtype=torch.float32, device=self.device)
-        for s in range(0, xf_rows.shape[0], chunk):
-            t = targets[s:s + chunk].contiguous()
-            _, out[s:s + chunk] = K.sample(self.lm_logits(xf_rows[s:s + chunk]), temperature, True, 0, forced=t)
-        return out

@@ -11,6 +11,7 @@ SwiGLU and (grouped-query) attention with head_dim 128:
 A file that names an ``architecture`` instead lists its layers one by one:
 
   Dulisun  chunked attention with a sink, mixtures of experts, output norms (``models/dulisun.py``); served only
+  Zafopel  latent attention beside the feed-forward, mixtures with scaled inputs, elementwise norms (``models/zafopel.py``); served only
 
 Anything the kernels do not implement is rejected here with a clear message (linear biases, attention
 dropout, other rope scaling types, head_dim != 128, sliding windows). Reference:
@@ -20,14 +21,16 @@ from __future__ import annotations
 
 import json
 from pathlib import Path
-from typing import Any, Dict, Mapping
+from typing import Any, Callable, Dict, List, Mapping, NamedTuple, Union
 
+from ..ops.kernels import LATENT_MAX_RANK
 from ..runtime.errors import RuntimeConfigError
 from .dulisun import AttentionMixer, DecoderLayer, DulisunConfig, DulisunModel, ExpertMixture
 from .llama import LlamaConfig, LlamaModel
+from .zafopel import DenseFF, InputScaledMixture, LatentMixer, ParallelLayer, ZafopelConfig, ZafopelModel
 
 FAMILIES = ("llama", "qwen3")
-ARCHITECTURES = ("Dulisun",)
+ServedConfig = Union[DulisunConfig, ZafopelConfig]
 
 
 def _llama3_rope_factor(cfg: Mapping[str, Any]) -> float:
@@ -118,13 +121,114 @@ def dulisun_config_dict(cfg: DulisunConfig) -> Dict[str, Any]:
     return {"architecture": "Dulisun", "vocab": cfg.vocab, "width": cfg.width, "norm": {"eps": cfg.norm_eps}, "layers": layers}
 
 
-def config_from_hf(hf: Mapping[str, Any], *, max_pos: int | None = None, lm_head: bool = True, scalar_head: bool = False) -> LlamaConfig | DulisunConfig:
+def _latent_mixer(kind: str, m: Mapping[str, Any], where: str, index: int, before: List[ParallelLayer]) -> LatentMixer:
+    """``latent_attention``: queries straight from the input, sliding window. ``latent_attention_2``: queries through a latent of their own,
+    causal, with a sink."""
+    second = kind == "latent_attention_2"
+    heads, dim, rot_dim, vdim, rank = (int(m[k]) for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank"))
+    rot = m["rot"]
+    if min(heads, dim, vdim, rank) < 1:
+        raise RuntimeConfigError(f"{where}: heads, dim, vdim and kv_rank must be at least 1")
+    if rot_dim < 0 or rot_dim % 2 or int(rot.get("dims", rot_dim)) != rot_dim:
+        raise RuntimeConfigError(f"{where}: the rotated part is rotated as a whole, so rot.dims must equal rot_dim and be even, got {rot.get('dims')}, {rot_dim}")
+    if rank > LATENT_MAX_RANK:
+        raise RuntimeConfigError(f"{where}: kv_rank {rank} is not supported (the attention kernels cover up to {LATENT_MAX_RANK})")
+    q_rank = int(m["q_rank"]) if second else 0
+    if second and not 1 <= q_rank <= 8192:
+        raise RuntimeConfigError(f"{where}: q_rank must lie in 1 to 8192, got {q_rank}")
+    mask = m.get("mask") or {}
+    window = 0 if second else int(mask.get("size", 0))
+    if not second and window < 1:
+        raise RuntimeConfigError(f"{where}: mask.size must be at least 1")
+    src = m.get("kv_from")
+    out = LatentMixer(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=rank, scale=float(m["scale"]), rot_base=float(rot["base"]),
+                      q_rank=q_rank, window=window, sink=second, kv_from=None if src is None else int(src))
+    if src is not None:
+        j = int(src)
+        if not 0 <= j < index or before[j].mixer.kv_from is not None:
+            raise RuntimeConfigError(f"{where}: kv_from must name an earlier layer with a latent of its own, got {j}")
+        o = before[j].mixer
+        if (o.kv_rank, o.rot_dim, o.rot_base) != (rank, rot_dim, out.rot_base):
+            raise RuntimeConfigError(f"{where}: kv_rank, rot_dim and rotation must equal those of layer {j}, whose latents it reads")
+    return out
+
+
+def _parallel_ff(m: Mapping[str, Any], where: str) -> DenseFF | InputScaledMixture:
+    kind = m.get("kind")
+    if kind == "dense":
+        if int(m["ff"]) < 1:
+            raise RuntimeConfigError(f"{where}: ff must be at least 1")
+        return DenseFF(int(m["ff"]))
+    if kind != "moe":
+        raise RuntimeConfigError(f"{where}: unsupported feed-forward kind {kind!r}; dense and moe are implemented")
+    e = InputScaledMixture(experts=int(m["router"]["experts"]), top=int(m["router"]["top"]), ff=int(m["expert"]["ff"]))
+    if e.ff < 1 or not 1 <= e.top <= e.experts:
+        raise RuntimeConfigError(f"{where}: cannot choose {e.top} of {e.experts} experts of size {e.ff}")
+    if e.experts > 1024:
+        raise RuntimeConfigError(f"{where}: {e.experts} experts exceed the kernels' limit of 1024")
+    return e
+
+
+def zafopel_config(cfg: Mapping[str, Any], max_pos: int | None = None) -> ZafopelConfig:
+    layers: List[ParallelLayer] = []
+    for i, l in enumerate(cfg["layers"]):
+        if l.get("type") not in ("latent_attention", "latent_attention_2"):
+            raise RuntimeConfigError(f"layer {i}: unsupported mixer type {l.get('type')!r}; latent_attention and latent_attention_2 are implemented")
+        mlp = l.get("mlp")
+        layers.append(ParallelLayer(_latent_mixer(l["type"], l["mixer"], f"layer {i} mixer", i, layers),
+                                    None if mlp is None else _parallel_ff(mlp, f"layer {i} mlp")))
+    if not layers:
+        raise RuntimeConfigError("the model has no layers")
+    return ZafopelConfig(width=int(cfg["width"]), vocab=int(cfg["vocab"]), layers=tuple(layers), norm_eps=float(cfg["norm"]["eps"]),
+                         max_pos=int(max_pos or 4096))
+
+
+def zafopel_config_dict(cfg: ZafopelConfig) -> Dict[str, Any]:
+    """The inverse of ``zafopel_config``."""
+    layers = []
+    for l in cfg.layers:
+        m, e = l.mixer, l.mlp
+        mixer: Dict[str, Any] = {"heads": m.heads, "dim": m.dim, "rot_dim": m.rot_dim, "vdim": m.vdim, "kv_rank": m.kv_rank, "scale": m.scale,
+                                 "rot": {"base": m.rot_base, "dims": m.rot_dim}}
+        if m.q_rank:
+            mixer["q_rank"] = m.q_rank
+        if m.window:
+            mixer["mask"] = {"size": m.window}
+        if m.kv_from is not None:
+            mixer["kv_from"] = m.kv_from
+        mlp: Dict[str, Any] | None = None
+        if isinstance(e, DenseFF):
+            mlp = {"kind": "dense", "ff": e.ff}
+        elif e is not None:
+            mlp = {"kind": "moe", "expert": {"ff": e.ff}, "router": {"experts": e.experts, "top": e.top}}
+        layers.append({"type": "latent_attention_2" if m.sink else "latent_attention", "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Zafopel", "vocab": cfg.vocab, "width": cfg.width, "norm": {"eps": cfg.norm_eps}, "layers": layers}
+
+
+class _Architecture(NamedTuple):
+    config: type
+    model: type
+    read: Callable[..., ServedConfig]
+    write: Callable[[Any], Dict[str, Any]]
+
+
+ARCHITECTURES: Dict[str, _Architecture] = {
+    "Dulisun": _Architecture(DulisunConfig, DulisunModel, dulisun_config, dulisun_config_dict),
+    "Zafopel": _Architecture(ZafopelConfig, ZafopelModel, zafopel_config, zafopel_config_dict),
+}
+
+
+def _architecture_of(cfg) -> _Architecture | None:
+    return next((a for a in ARCHITECTURES.values() if isinstance(cfg, a.config)), None)
+
+
+def config_from_hf(hf: Mapping[str, Any], *, max_pos: int | None = None, lm_head: bool = True, scalar_head: bool = False) -> LlamaConfig | ServedConfig:
     if "architecture" in hf:
         if hf["architecture"] not in ARCHITECTURES:
             raise RuntimeConfigError(f"unsupported architecture {hf['architecture']!r}; supported: {', '.join(ARCHITECTURES)}")
         if scalar_head or not lm_head:
             raise RuntimeConfigError(f"{hf['architecture']} models have a language-model head only")
-        return dulisun_config(hf, max_pos)
+        return ARCHITECTURES[hf["architecture"]].read(hf, max_pos)
     family = hf.get("model_type")
     if family not in FAMILIES:
         raise RuntimeConfigError(f"unsupported model_type {family!r}; supported: {', '.join(FAMILIES)}")
@@ -151,7 +255,7 @@ def config_from_hf(hf: Mapping[str, Any], *, max_pos: int | None = None, lm_head
         rope_scaling_factor=_llama3_rope_factor(hf) if family == "llama" else 1.0, family=family)
 
 
-def config_from_hf_path(path, **kw) -> LlamaConfig | DulisunConfig:
+def config_from_hf_path(path, **kw) -> LlamaConfig | ServedConfig:
     p = Path(path)
     cfg_file = p / "config.json" if p.is_dir() else p
     if not cfg_file.exists():
@@ -161,7 +265,8 @@ def config_from_hf_path(path, **kw) -> LlamaConfig | DulisunConfig:
 
 def model_class(cfg):
     """The model class that runs a configuration."""
-    return DulisunModel if isinstance(cfg, DulisunConfig) else LlamaModel
+    arch = _architecture_of(cfg)
+    return LlamaModel if arch is None else arch.model
 
 
 def load_model(path, device, *, dtype=None, max_pos: int | None = None):
@@ -178,15 +283,16 @@ def load_model(path, device, *, dtype=None, max_pos: int | None = None):
         raise RuntimeConfigError(f"{cfg.family} models run in bfloat16 only")
     if torch.device(device).type == "cuda":
         _lib.ensure(cls.KERNEL_SOURCES)
-    model = cls(cfg, device, dtype=dtype, seed=None) if cls is DulisunModel else cls(cfg, device)
+    model = cls(cfg, device) if cls is LlamaModel else cls(cfg, device, dtype=dtype, seed=None)
     load_weights(model, path)
     return model
 
 
 def hf_config_dict(cfg) -> Dict[str, Any]:
     """The inverse mapping (used when exporting a checkpoint next to its architecture)."""
-    if isinstance(cfg, DulisunConfig):
-        return dulisun_config_dict(cfg)
+    arch = _architecture_of(cfg)
+    if arch is not None:
+        return arch.write(cfg)
     out: Dict[str, Any] = {
         "model_type": cfg.family, "hidden_size": cfg.d_model, "intermediate_size": cfg.d_ff, "num_hidden_layers": cfg.n_layers,
         "num_attention_heads": cfg.n_heads, "num_key_value_heads": cfg.n_kv_heads, "head_dim": cfg.head_dim, "vocab_size": cfg.vocab,

@@ -88,11 +88,21 @@ _SIGNATURES = {
     "rpeg_rotary_append": [P, I, LL, I, I, I, I, P, P, P, P, P, I, P, I, P, P, I, I, I, I, I, I, I, F, I, P],
     "rpeg_rows_attn": [P, I, P, P, P, I, P, P, P, P, P, I, P, P, I, I, I, I, I, I, F, I, P, P],
     "rpeg_window_prefill": [P, I, P, P, LL, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P],
-    "rpeg_moe_route": [P, I, LL, I, I, I, I, I, I, I, P, P, P, P, P],
-    "rpeg_moe_dispatch": [P, I, P, P, P, I, I, I, P, P, P, I, P],
+    "rpeg_moe_route": [P, I, LL, I, I, I, I, I, I, I, I, P, P, P, P, P],
+    "rpeg_moe_dispatch": [P, I, P, P, P, P, I, I, I, P, P, P, I, P],
     "rpeg_moe_gemm": [P, LL, P, P, P, P, I, I, I, LL, I, I, I, I, I, I, I, I, P, P],
     "rpeg_moe_gemm_f32": [P, P, P, P, P, I, I, I, I, I, I, I, I, I, P],
     "rpeg_gemm_f32": [P, P, P, I, I, I, I, I, I, P],
+    "rpeg_gemm_f32_batched": [P, P, P, I, I, I, I, I, I, LL, LL, LL, I, I, P],
+    "rpeg_stream_update": [I, P, I, LL, I, P, I, P, I, LL, I, P, P, I, I, LL, P, P, P, P, P, I, I, I, P],
+    "rpeg_latent_rows": [P, I, LL, I, I, P, P, P, P, I, I, F, I, I, I, P, P, I, I, I, P, P, P, I, I, I, I, P, I, P, I, I, I, P],
+    "rpeg_latent_gather": [P, I, P, I, P, P, P, P, I, I, P, P],
+    "rpeg_latent_attn_rows": [P, P, P, I, P, P, P, P, P, I, I, I, I, I, F, I, P],
+    "rpeg_latent_decode_ctas": [I, I],
+    "rpeg_latent_decode": [P, P, LL, P, I, P, P, P, P, P, P, I, I, I, I, I, I, F, P, P],
+    "rpeg_latent_prefill_fits": [I, I, I],
+    "rpeg_latent_prefill": [P, I, I, P, P, LL, I, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P, P],
+    "rpeg_head_gemm": [P, P, P, I, I, I, I, I, I, I, I, I, P, P],
     "rpeg_flash_attn_fwd": [P, I, I, I, I, P, I, I, I, I, I, I, F, P, P, P, P],
     "rpeg_flash_attn_bwd": [P, I, I, I, I, P, P, P, P, I, I, I, I, I, I, F, P, P, P, I, P, P],
 }
@@ -133,6 +143,9 @@ def lib() -> ctypes.CDLL:
         if hasattr(handle, "rpeg_rows_attn_scratch"):
             handle.rpeg_rows_attn_scratch.argtypes = [I, I, I, I]
             handle.rpeg_rows_attn_scratch.restype = c_longlong
+        if hasattr(handle, "rpeg_latent_decode_scratch"):
+            handle.rpeg_latent_decode_scratch.argtypes = [I, I, I, I]
+            handle.rpeg_latent_decode_scratch.restype = c_longlong
         _lib = handle
     return _lib
 

@@ -429,6 +429,10 @@ class Partials:
     def stride(self) -> int:
         return self.M * self.N
 
+    def columns(self, c0: int) -> "Partials":
+        """The same partials seen from column ``c0`` on (the row pitch stays ``N``)."""
+        return Partials(self.buf[c0:], self.splits, self.M, self.N)
+
     def reduce(self) -> torch.Tensor:
         return self.buf[: self.splits * self.stride].view(self.splits, self.M, self.N).sum(0)
 
@@ -653,11 +657,12 @@ _NORM_ACT, _NORM_PARTIALS, _NORM_MOE, _NORM_EMBED, _NORM_STREAM = range(5)
 
 
 class MoEOutput:
-    """Expert outputs of ``T`` tokens before their weighted sum: ``y`` rows in segment order, ``row_of`` / ``weights`` ``[T, top]``."""
+    """Expert outputs of ``T`` tokens before their sum: ``y`` rows in segment order, ``row_of`` / ``weights`` ``[T, top]`` (weights None:
+    a plain sum)."""
 
     __slots__ = ("y", "row_of", "weights", "top", "n_shared")
 
-    def __init__(self, y: torch.Tensor, row_of: torch.Tensor, weights: torch.Tensor, n_shared: int):
+    def __init__(self, y: torch.Tensor, row_of: torch.Tensor, weights: torch.Tensor | None, n_shared: int):
         self.y, self.row_of, self.weights, self.n_shared = y, row_of, weights, n_shared
         self.top = row_of.shape[1]
 
@@ -781,8 +786,9 @@ class MoERouting:
         self.ids, self.weights, self.row_of, self.seg_off, self.x_sorted, self.x = ids, weights, row_of, seg_off, x_sorted, x
 
 
-def moe_route(logits, n_experts: int, top: int, counts: torch.Tensor, *, n_groups: int = 1, keep_groups: int = 1, renormalize: bool = False):
-    """Softmax routing of ``logits`` (fp32 ``[T, >= E]`` or ``Partials``): the ``top`` largest scores among the experts of the
+def moe_route(logits, n_experts: int, top: int, counts: torch.Tensor, *, n_groups: int = 1, keep_groups: int = 1, renormalize: bool = False,
+              sigmoid: bool = False):
+    """Softmax (or ``sigmoid``) routing of ``logits`` (fp32 ``[T, >= E]`` or ``Partials``): the ``top`` largest scores among the experts of the
     ``keep_groups`` best of ``n_groups`` equal groups. ``counts [E]`` int32 must be zero; every choice takes a ticket there.
     Returns ``(ids, weights, tickets)``, each ``[T, top]``."""
     part = isinstance(logits, Partials)
@@ -795,13 +801,14 @@ def moe_route(logits, n_experts: int, top: int, counts: torch.Tensor, *, n_group
     ids, ticket = torch.empty((rows, top), **i32), torch.empty((rows, top), **i32)
     wts = torch.empty((rows, top), dtype=torch.float32, device=buf.device)
     check(lib().rpeg_moe_route(buf.data_ptr(), logits.splits if part else 1, logits.stride if part else 0, ld, rows, n_experts, n_groups, keep_groups,
-                               top, int(renormalize), ids.data_ptr(), wts.data_ptr(), ticket.data_ptr(), counts.data_ptr(), _stream()),
+                               top, int(renormalize), int(sigmoid), ids.data_ptr(), wts.data_ptr(), ticket.data_ptr(), counts.data_ptr(), _stream()),
           "rpeg_moe_route")
     return ids, wts, ticket
 
 
-def moe_dispatch(x: torch.Tensor, ids, wts, ticket, counts, n_experts: int) -> MoERouting:
-    """Copy every token's row into the segments of its experts."""
+def moe_dispatch(x: torch.Tensor, ids, wts, ticket, counts, n_experts: int, *, weigh_inputs: bool = False) -> MoERouting:
+    """Copy every token's row into the segments of its experts; ``weigh_inputs``: multiplied by the choice's weight there (the
+    outputs are then summed as they are)."""
     rows, dp = x.shape
     top = ids.shape[1]
     if not x.is_contiguous():
@@ -809,17 +816,22 @@ def moe_dispatch(x: torch.Tensor, ids, wts, ticket, counts, n_experts: int) -> M
     row_of = torch.empty_like(ids)
     seg_off = torch.empty(n_experts + 1, dtype=torch.int32, device=x.device)
     xs = torch.empty((rows * top, dp), dtype=x.dtype, device=x.device)
-    check(lib().rpeg_moe_dispatch(x.data_ptr(), dp, ids.data_ptr(), ticket.data_ptr(), counts.data_ptr(), rows, n_experts, top, xs.data_ptr(),
+    check(lib().rpeg_moe_dispatch(x.data_ptr(), dp, ids.data_ptr(), ticket.data_ptr(), _ptr(wts if weigh_inputs else None), counts.data_ptr(), rows, n_experts, top, xs.data_ptr(),
                                   row_of.data_ptr(), seg_off.data_ptr(), int(x.dtype == torch.float32), _stream()), "rpeg_moe_dispatch")
-    return MoERouting(ids, wts, row_of, seg_off, xs, x)
+    return MoERouting(ids, None if weigh_inputs else wts, row_of, seg_off, xs, x)
+
+
+FF_ACTS = {"none": 0, "gelu": 1, "swiglu": 2, "relu2": 3}
 
 
 def moe_gemm(a: torch.Tensor, b: torch.Tensor, r: MoERouting, n_experts: int, n_shared: int, *, shared_x: torch.Tensor | None = None,
-             gelu: bool = False, bn: int = 0) -> torch.Tensor:
-    """``C[rows of segment s] = act(a[rows of s] @ b[s].T)`` over the experts' segments; ``b [E + n_shared, N, K]``. The always-on
-    segments take their rows from ``shared_x [T, K]`` (tokens in order) or, without it, from ``a`` behind the routed rows."""
+             act: str = "none", bn: int = 0) -> torch.Tensor:
+    """``C[rows of segment s] = act(a[rows of s] @ b[s].T)`` over the experts' segments; ``b [E + n_shared, N, K]``. ``act``: none, gelu,
+    relu2 (squared relu) or swiglu (``b [E + n_shared, 2 N, K]``, gate rows first: ``silu(gate) * up``). The always-on segments take their rows from ``shared_x [T, K]`` (tokens in order) or, without it, from ``a`` behind the routed rows."""
     T, top = r.row_of.shape
     S, N, Kd = b.shape
+    code = FF_ACTS[act]
+    N = N // 2 if act == "swiglu" else N
     if S != n_experts + n_shared or a.shape[1] != Kd or not b.is_contiguous() or a.stride(1) != 1:
         raise ValueError("moe_gemm: operand shapes do not fit the segments")
     need = T * top + (0 if shared_x is not None else n_shared * T)
@@ -830,10 +842,219 @@ def moe_gemm(a: torch.Tensor, b: torch.Tensor, r: MoERouting, n_experts: int, n_
         if shared_x is not None and shared_x.stride(0) != a.stride(0):
             raise ValueError("moe_gemm: both operands need one row pitch")
         check(lib().rpeg_moe_gemm_f32(a.data_ptr(), _ptr(shared_x), b.data_ptr(), c.data_ptr(), r.seg_off.data_ptr(), n_experts, n_shared, T, N, Kd,
-                                      a.stride(0), Kd, c.stride(0), int(gelu), _stream()), "rpeg_moe_gemm_f32")
+                                      a.stride(0), Kd, c.stride(0), code, _stream()), "rpeg_moe_gemm_f32")
         return c
     _req(a, torch.bfloat16, "a")
     check(lib().rpeg_moe_gemm(a.data_ptr(), a.shape[0], _ptr(shared_x), b.data_ptr(), c.data_ptr(), r.seg_off.data_ptr(), n_experts, n_shared, T,
-                              T * top, N, Kd, a.stride(0), 0 if shared_x is None else shared_x.stride(0), Kd, c.stride(0), int(gelu), bn,
+                              T * top, N, Kd, a.stride(0), 0 if shared_x is None else shared_x.stride(0), Kd, c.stride(0), code, bn,
                               status_word(a.device).data_ptr(), _stream()), "rpeg_moe_gemm")
     return c
+
+
+_ZERO_SEGMENT: dict[torch.device, torch.Tensor] = {}
+
+
+def ff_first(x: torch.Tensor, w: torch.Tensor, act: str) -> torch.Tensor:
+    """``act(x @ w.T)``, the first product of a dense feed-forward with its activation in the epilogue (``act`` and the layout of ``w``
+    as in ``moe_gemm``): a mixture of one always-on expert."""
+    if x.device not in _ZERO_SEGMENT:
+        _ZERO_SEGMENT[x.device] = torch.zeros(1, dtype=torch.int32, device=x.device)
+    r = MoERouting(None, None, torch.empty((x.shape[0], 0), dtype=torch.int32, device=x.device), _ZERO_SEGMENT[x.device], x, x)
+    return moe_gemm(x, w.unsqueeze(0), r, 0, 1, shared_x=x, act=act)
+
+
+# --------------------------------------------------------------------------- stream of parallel sublayers
+def stream_update(a, b, alpha: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, x: torch.Tensor, *, ids: torch.Tensor | None = None) -> torch.Tensor:
+    """``x += a + b`` on the fp32 stream ``x [T, dp]``, returns ``tanh(alpha * x) * w + bias`` in the dtype of ``w``. ``a``: an activation
+    ``[T, >= dp]``, ``Partials``, or an embedding table whose rows ``ids`` become ``x``; ``b``: None, an activation, ``Partials`` or a
+    ``MoEOutput``. ``alpha``: fp32 scalar on the device."""
+    dp, rows = w.numel(), x.shape[0]
+    f32 = w.dtype == torch.float32
+    if x.dtype != torch.float32 or x.shape != (rows, dp) or not x.is_contiguous() or bias.dtype != w.dtype or bias.numel() != dp:
+        raise ValueError("stream_update: the stream must be a contiguous fp32 [T, dp] tensor, w and bias [dp]")
+    _req(alpha, torch.float32, "alpha")
+
+    def source(s):
+        """(kind, tensor, splits, stride, row pitch)"""
+        if s is None:
+            return -1, None, 1, 0, 0
+        if isinstance(s, Partials):
+            n, out = s.M, (_NORM_PARTIALS, s.buf, s.splits, s.stride, s.N)
+        elif isinstance(s, MoEOutput):
+            n, out = s.row_of.shape[0], (_NORM_MOE, s.y, 1, 0, s.y.stride(0))
+        else:
+            n, out = rows if ids is not None else s.shape[0], (_NORM_EMBED if ids is not None else _NORM_ACT, s, 1, 0, s.stride(0))
+        if n != rows or out[4] < dp or out[1].dtype != (torch.float32 if isinstance(s, Partials) else w.dtype):
+            raise ValueError("stream_update: a source does not fit the stream or the weights' dtype")
+        return out
+
+    if ids is not None:
+        _req(ids, torch.int32, "ids")
+        if ids.numel() != rows:
+            raise ValueError("stream_update: one id per row")
+        if _chk.active():
+            _chk.embed("rpeg_stream_update", ids, a.shape[0])
+    ka, ta, pa, sa, la = source(a)
+    kb, tb, pb, sb, lb = source(b)
+    moe = isinstance(b, MoEOutput)
+    y = torch.empty((rows, dp), dtype=w.dtype, device=w.device)
+    check(lib().rpeg_stream_update(ka, ta.data_ptr(), pa, sa, la, _ptr(ids), kb, _ptr(tb), pb, sb, lb, _ptr(b.row_of if moe else None),
+                                   _ptr(b.weights if moe else None), b.top if moe else 0, b.n_shared if moe else 0, rows * b.top if moe else 0,
+                                   alpha.data_ptr(), w.data_ptr(), bias.data_ptr(), x.data_ptr(), y.data_ptr(), rows, dp, int(f32), _stream()),
+          "rpeg_stream_update")
+    return y
+
+
+# --------------------------------------------------------------------------- latent attention
+LATENT_MAX_RANK = 1024           # latent width the kernels cover
+
+
+def head_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, transposed: bool = False) -> torch.Tensor:
+    """``out[:, h] = a[:, h] @ w[h].T`` for every head (``transposed``: ``@ w[h]``); ``a [T, H, K]`` and ``out [T, H, N]`` may be strided
+    views with contiguous last dimensions, ``w [H, N, K]`` (``[H, K, N]``) is contiguous."""
+    T, H, Kd = a.shape
+    N = out.shape[2]
+    if w.shape != ((H, Kd, N) if transposed else (H, N, Kd)) or out.shape[:2] != (T, H) or a.stride(2) != 1 or out.stride(2) != 1 or not w.is_contiguous():
+        raise ValueError("head_gemm: operand shapes do not fit")
+    if not a.dtype == w.dtype == out.dtype:
+        raise TypeError("head_gemm: operands must share a dtype")
+    if a.dtype == torch.float32:
+        check(lib().rpeg_gemm_f32_batched(a.data_ptr(), w.data_ptr(), out.data_ptr(), T, N, Kd, a.stride(0), N if transposed else Kd, out.stride(0),
+                                          a.stride(1), N * Kd, out.stride(1), H, int(transposed), _stream()), "rpeg_gemm_f32_batched")
+        return out
+    _req(a, torch.bfloat16, "a")
+    check(lib().rpeg_head_gemm(a.data_ptr(), w.data_ptr(), out.data_ptr(), T, N, Kd, H, a.stride(0), a.stride(1), out.stride(0), out.stride(1),
+                               int(transposed), status_word(a.device).data_ptr(), _stream()), "rpeg_head_gemm")
+    return out
+
+
+def latent_rows(src, pos, slot, cos_t, sin_t, rot: int, rot_p: int, eps: float, *, q_latent=None, kv=None, queries=None) -> None:
+    """Between a projection and latent attention, any of (column numbers refer to ``src``, an activation or ``Partials``):
+      q_latent  (column, true width, weight, out [T, width_p]): weighted RMS norm of a query latent
+      kv        (column, true rank, weight, cache [pages, 1, PAGE, rank_p + rot_p], page_table): the normed latent and the rotated shared key
+                part of every token into its cache row
+      queries   (column, heads, dim_p, out or None, rotated [T, H, rot_p]): heads of ``[dim_p | rot_p]`` columns; the rotated parts go to the
+                (strided) view ``rotated``, which may be their place in ``src``; the others to ``out [T, H * dim_p]``, if given."""
+    part = isinstance(src, Partials)
+    rows, ld = (src.M, src.N) if part else (src.shape[0], src.stride(0))
+    ref = next(t for t in (q_latent and q_latent[3], kv and kv[3], queries and queries[4]) if t is not None)
+    f32 = ref.dtype == torch.float32
+    if (part and f32) or (not part and src.dtype != ref.dtype):
+        raise TypeError("latent_rows: source and outputs must share a dtype (split-K partials belong to the bf16 path)")
+    if rot and (cos_t.shape[1] * 2 != rot or cos_t.shape != sin_t.shape):
+        raise ValueError("latent_rows: the tables do not fit the rotated width")
+    nq = (0, 0, 0, None, None)
+    if q_latent is not None:
+        c0, n, w, out = q_latent
+        if not out.is_contiguous() or out.shape != (rows, w.numel()):
+            raise ValueError("latent_rows: the query latent's buffer must be [T, width]")
+        nq = (c0, n, w.numel(), w.data_ptr(), out.data_ptr())
+    lat = (0, 0, 0, None, None, None, 0)
+    if kv is not None:
+        c0, n, w, cache, table = kv
+        if cache.shape[1] != 1 or cache.shape[3] != w.numel() + rot_p:
+            raise ValueError("latent_rows: the cache does not fit the latent")
+        if _chk.active():
+            _chk.kv_append("rpeg_latent_rows", rows, slot, pos, table, cache, 1, cache.shape[3], cos_t if rot else None)
+        lat = (c0, n, w.numel(), w.data_ptr(), cache.data_ptr(), table.data_ptr(), table.stride(0))
+    qs = (0, 0, 0, None, 0, None, 0, 0)
+    if queries is not None:
+        c0, H, dim_p, out, rotated = queries
+        if rotated.shape != (rows, H, rot_p) or (rot_p and rotated.stride(2) != 1) or (out is not None and (out.shape != (rows, H * dim_p) or not out.is_contiguous())):
+            raise ValueError("latent_rows: the query buffers do not fit")
+        if rot and _chk.active():
+            _chk.rope("rpeg_latent_rows", pos, rows, cos_t)
+        qs = (c0, H, dim_p, _ptr(out), H * dim_p, rotated.data_ptr(), rotated.stride(0), rotated.stride(1))
+    check(lib().rpeg_latent_rows((src.buf if part else src).data_ptr(), src.splits if part else 0, src.stride if part else 0, ld, rows, pos.data_ptr(),
+                                 slot.data_ptr(), _ptr(cos_t), _ptr(sin_t), rot, rot_p, eps, *nq, *lat, *qs, int(f32), _stream()), "rpeg_latent_rows")
+
+
+def latent_gather(cache: torch.Tensor, page_table, slot, cu, off, lo, rows: int) -> torch.Tensor:
+    """The cache rows packed requests see, ``[rows, W]``: rows ``off[b] .. off[b + 1]`` are the positions from ``lo[b]`` on of page-table row
+    ``slot[cu[b]]``."""
+    W = cache.shape[3]
+    out = torch.empty((rows, W), dtype=cache.dtype, device=cache.device)
+    if _chk.active():
+        _chk.packed_sequences("rpeg_latent_gather", off, rows, rows)
+        _chk.paged_attention("rpeg_latent_gather", lo.numel(), lo + off[1:] - off[:-1], page_table[slot[cu[:-1].long()].long()], cache, 1, W)
+    check(lib().rpeg_latent_gather(cache.data_ptr(), W * cache.element_size(), page_table.data_ptr(), page_table.stride(0), slot.data_ptr(), cu.data_ptr(),
+                                   off.data_ptr(), lo.data_ptr(), lo.numel(), rows, out.data_ptr(), _stream()), "rpeg_latent_gather")
+    return out
+
+
+def latent_attn_rows(q: torch.Tensor, cache: torch.Tensor, rank_p: int, page_table, slot, pos, *, window: int = 0, scale: float, lens=None,
+                     sink: torch.Tensor | None = None) -> torch.Tensor:
+    """Latent attention of single query rows ``q [T, H, W]`` over the cache rows of page-table row ``slot[t]``: row ``t`` at position ``p =
+    pos[t]`` (or ``lens[t] - 1``; ``lens[t] = 0``: nothing, the row is zero) sees the last ``window`` positions up to its own (0: all). Returns
+    the averaged latents ``[T, H, rank_p]``. ``sink [H]`` fp32 joins the softmax denominator. CUDA cores, bf16 or fp32."""
+    T, H, W = q.shape
+    if q.dtype != cache.dtype or not q.is_contiguous() or cache.shape[3] != W:
+        raise TypeError("latent_attn_rows: q must be contiguous [T, H, W] in the cache's dtype")
+    if _chk.active():
+        _chk.paged_attention("rpeg_latent_attn_rows", T, (pos + 1) if lens is None else lens, page_table[slot[:T].long()], cache, 1, W)
+    out = torch.empty((T, H, rank_p), dtype=q.dtype, device=q.device)
+    check(lib().rpeg_latent_attn_rows(q.data_ptr(), cache.data_ptr(), page_table.data_ptr(), page_table.stride(0), slot.data_ptr(), pos.data_ptr(),
+                                      _ptr(lens), _ptr(sink), out.data_ptr(), T, H, rank_p, W, window, scale, int(q.dtype == torch.float32), _stream()),
+          "rpeg_latent_attn_rows")
+    return out
+
+
+def latent_decode_ctas_per_sm(rank_p: int, width: int) -> int:
+    """CTAs of ``latent_decode`` an SM holds (0: sizes it does not cover)."""
+    return int(lib().rpeg_latent_decode_ctas(rank_p, width))
+
+
+def latent_decode_fits(rank_p: int, width: int) -> bool:
+    return latent_decode_ctas_per_sm(rank_p, width) > 0
+
+
+def latent_decode_scratch(rows: int, n_heads: int, rank_p: int, nsplit: int) -> int:
+    """fp32 elements of split scratch ``latent_decode`` needs."""
+    return int(lib().rpeg_latent_decode_scratch(rows, n_heads, rank_p, nsplit))
+
+
+def latent_decode(q: torch.Tensor, cache: torch.Tensor, rank_p: int, page_table, slot, pos, *, window: int = 0, scale: float, lens=None,
+                  sink: torch.Tensor | None = None, nsplit: int = 1, scratch: torch.Tensor | None = None) -> torch.Tensor:
+    """``latent_attn_rows`` on the tensor cores (bf16; sizes as ``latent_decode_fits``). The cache must hold finite numbers everywhere.
+    ``nsplit > 1``: every row's pages are shared by that many CTAs (``scratch`` as ``latent_decode_scratch``)."""
+    _req(q, torch.bfloat16, "q")
+    _req(cache, torch.bfloat16, "cache")
+    T, H, W = q.shape
+    if not q.is_contiguous() or cache.shape[1:] != (1, KV_PAGE, W):
+        raise ValueError("latent_decode: q must be contiguous [T, H, W], the cache [pages, 1, PAGE, W]")
+    if nsplit > 1 and (scratch is None or scratch.numel() < latent_decode_scratch(T, H, rank_p, nsplit)):
+        raise ValueError("latent_decode: split attention needs scratch")
+    if _chk.active():
+        _chk.paged_attention("rpeg_latent_decode", T, (pos + 1) if lens is None else lens, page_table[slot[:T].long()], cache, 1, W)
+    out = torch.empty((T, H, rank_p), dtype=torch.bfloat16, device=q.device)
+    check(lib().rpeg_latent_decode(q.data_ptr(), cache.data_ptr(), cache.shape[0], page_table.data_ptr(), page_table.stride(0), slot.data_ptr(), pos.data_ptr(),
+                                   _ptr(lens), _ptr(sink), out.data_ptr(), _ptr(scratch), T, H, rank_p, W, window, nsplit, scale,
+                                   status_word(q.device).data_ptr(), _stream()), "rpeg_latent_decode")
+    return out
+
+
+def latent_prefill_fits(dim_p: int, rot_p: int, vdim_p: int) -> bool:
+    """Head sizes ``latent_prefill`` covers (padded): unrotated and rotated parts up to three runs of 64 together, values up to 128."""
+    return bool(lib().rpeg_latent_prefill_fits(dim_p, rot_p, vdim_p))
+
+
+def latent_prefill(q: torch.Tensor, kv: torch.Tensor, rows: torch.Tensor, dim_p: int, vdim_p: int, rank_p: int, cu, pos, off, lo, max_len: int, *,
+                   window: int = 0, scale: float, sink: torch.Tensor | None = None) -> torch.Tensor:
+    """Prompt attention of packed portions (request ``b`` owns query rows ``cu[b] .. cu[b + 1]`` at consecutive positions ``pos``) over formed keys
+    and values: ``q [T, H, dim_p + rot_p]`` (may be strided), ``kv [n, H * dim_p + H * vdim_p]`` from the gathered cache rows ``rows [n, W]``, of
+    which request ``b`` sees ``off[b] .. off[b + 1]``, positions ``lo[b]`` on. Visibility as in ``latent_attn_rows``. Returns
+    ``[T, H * vdim_p]``. bf16, ``scale > 0``."""
+    for t, name in ((q, "q"), (kv, "kv"), (rows, "rows")):
+        _req(t, torch.bfloat16, name)
+    T, H, hw = q.shape
+    n, W = rows.shape
+    if q.stride(2) != 1 or kv.shape != (n, H * (dim_p + vdim_p)) or not kv.is_contiguous() or not rows.is_contiguous() or hw - dim_p != W - rank_p:
+        raise ValueError("latent_prefill: operand shapes do not fit")
+    if _chk.active():
+        _chk.packed_sequences("rpeg_latent_prefill", cu, T, max_len)
+        _chk.packed_sequences("rpeg_latent_prefill", off, n, n)
+    out = torch.empty((T, H * vdim_p), dtype=torch.bfloat16, device=q.device)
+    check(lib().rpeg_latent_prefill(q.data_ptr(), q.stride(0), q.stride(1), kv.data_ptr(), rows.data_ptr(), n, W, rank_p, cu.data_ptr(), pos.data_ptr(),
+                                    off.data_ptr(), lo.data_ptr(), _ptr(sink), out.data_ptr(), out.stride(0), T, cu.numel() - 1, max_len, H, dim_p,
+                                    hw - dim_p, vdim_p, window, scale, status_word(q.device).data_ptr(), _stream()), "rpeg_latent_prefill")
+    return out

@@ -157,26 +157,40 @@ def load_hf_weights(model, model_dir) -> int:
     return copied
 
 
+class _Checkpoint:
+    """Tensors of a directory by name, with their shapes checked and the unread ones remembered."""
+
+    def __init__(self, model, model_dir):
+        self.dir, self.model = model_dir, model
+        self.index = _open_shards(model_dir)
+        self.used: set = set()
+        self.copied = 0
+
+    def get(self, name: str, *shape: int, dtype=None):
+        if name not in self.index:
+            raise RuntimeConfigError(f"tensor {name} is missing from {self.dir}")
+        t = self.index[name].get_tensor(name)
+        if tuple(t.shape) != shape:
+            raise RuntimeConfigError(f"shape mismatch of {name}: checkpoint {tuple(t.shape)} vs model {shape}")
+        self.used.add(name)
+        self.copied += t.numel()
+        return t.to(device=self.model.device, dtype=dtype or self.model.dtype)
+
+    def finish(self) -> int:
+        """Warn about tensors without a place; the number of parameters copied."""
+        left = sorted(set(self.index) - self.used)
+        if left:
+            warnings.warn(f"{self.dir} holds {len(left)} tensors this model has no place for: {', '.join(left[:5])}", stacklevel=3)
+        return self.copied
+
+
 def load_dulisun_weights(model, model_dir) -> int:
     """Copy a Dulisun checkpoint into ``model``: linear weights are ``[out, in]`` under ``l<i>.mix.*`` and ``l<i>.mlp.*``,
     queries and keys are stacked, experts become the segments of one grouped matrix. Tensors without a place are reported
     as a warning. Returns the number of parameters copied."""
     cfg = model.cfg
-    idx = _open_shards(model_dir)
-    used = set()
-    copied = 0
-
-    def get(name: str, *shape: int):
-        nonlocal copied
-        if name not in idx:
-            raise RuntimeConfigError(f"tensor {name} is missing from {model_dir}")
-        t = idx[name].get_tensor(name)
-        if tuple(t.shape) != shape:
-            raise RuntimeConfigError(f"shape mismatch of {name}: checkpoint {tuple(t.shape)} vs model {shape}")
-        used.add(name)
-        copied += t.numel()
-        return t.to(device=model.device, dtype=model.dtype)
-
+    c = _Checkpoint(model, model_dir)
+    get = c.get
     d = cfg.width
     model.p["embed"][: cfg.vocab, :d].copy_(get("embed", cfg.vocab, d))
     model.p["embed_norm"][:d].copy_(get("embed.norm", d))
@@ -194,15 +208,56 @@ def load_dulisun_weights(model, model_dir) -> int:
             if e.shared_ff:
                 model.put_shared(i, get(f"l{i}.mlp.shared.up", e.shared_ff, d), get(f"l{i}.mlp.shared.down", d, e.shared_ff))
             model.p[f"l{i}.norm2"][:d].copy_(get(f"l{i}.norm2", d))
-    left = sorted(set(idx) - used)
-    if left:
-        warnings.warn(f"{model_dir} holds {len(left)} tensors this model has no place for: {', '.join(left[:5])}", stacklevel=2)
-    return copied
+    return c.finish()
+
+
+def load_zafopel_weights(model, model_dir) -> int:
+    """Copy a Zafopel checkpoint into ``model`` (names as in ``load_dulisun_weights``): everything that reads the layer's input through the
+    attention's side is stacked with the router, the key and value maps are stacked, experts become the segments of grouped matrices."""
+    import torch
+    cfg = model.cfg
+    c = _Checkpoint(model, model_dir)
+    get = c.get
+    d = cfg.width
+
+    def norm(i: int, name: str) -> None:
+        model.put_norm(i, get(name + ".alpha", dtype=torch.float32), get(name, d), get(name + ".b", d))
+
+    model.p["embed"][: cfg.vocab, :d].copy_(get("embed", cfg.vocab, d))
+    model.p["head"][: cfg.vocab, :d].copy_(get("head", cfg.vocab, d))
+    norm(cfg.n_layers, "final.norm")
+    for i, layer in enumerate(cfg.layers):
+        m, e = layer.mixer, layer.mlp
+        norm(i, f"l{i}.norm1")
+        pre = f"l{i}.mix."
+        q_rows = m.heads * (m.dim + m.rot_dim)
+        if m.q_rank:
+            model.put_query_latent(i, get(pre + "dq", m.q_rank, d), get(pre + "dq.norm", m.q_rank))
+            model.put_q(i, get(pre + "uq", q_rows, m.q_rank))
+        else:
+            model.put_q(i, get(pre + "q", q_rows, d))
+        if m.kv_from is None:
+            model.put_latent(i, get(pre + "dkv", m.kv_rank + m.rot_dim, d), get(pre + "dkv.norm", m.kv_rank))
+        model.put_kv_maps(i, get(pre + "uk", m.heads * m.dim, m.kv_rank), get(pre + "uv", m.heads * m.vdim, m.kv_rank))
+        model.put_o(i, get(pre + "o", d, m.heads * m.vdim))
+        if m.sink:
+            model.sink[i].copy_(get(pre + "sink", m.heads, dtype=torch.float32))
+        pre = f"l{i}.mlp."
+        if e is not None and hasattr(e, "experts"):
+            model.put_router(i, get(pre + "router", e.experts, d))
+            for s in range(e.experts):
+                model.put_expert(i, s, get(f"{pre}e{s}.gate", e.ff, d), get(f"{pre}e{s}.up", e.ff, d), get(f"{pre}e{s}.down", d, e.ff))
+        elif e is not None:
+            model.put_dense(i, get(pre + "up", e.ff, d), get(pre + "down", d, e.ff))
+    return c.finish()
+
+
+_LOADERS = {"dulisun": load_dulisun_weights, "zafopel": load_zafopel_weights}
 
 
 def load_weights(model, model_dir) -> int:
     """Load a checkpoint with the naming of the model's family."""
-    return (load_dulisun_weights if getattr(model.cfg, "family", "") == "dulisun" else load_hf_weights)(model, model_dir)
+    return _LOADERS.get(getattr(model.cfg, "family", ""), load_hf_weights)(model, model_dir)
 
 
 def save_hf_weights(model, model_dir, shard_bytes: int = 4 << 30) -> None:
