@@ -225,8 +225,9 @@ def main() -> None:
                          "tcgen05 kernel) instead of once per row through L2; off by default: measured slower on the full step")
     ap.add_argument("--budget-s", type=float, default=420.0,
                     help="wall-clock budget for warm-up plus timed steps; the timed step count is cut to fit and reported")
-    ap.add_argument("--serve", action="store_true", help="instead of the RLHF iteration: prefill and decode throughput of the Dulisun family "
-                    "beside the Llama family at equal size, with every kernel's distance from its roofline (one GPU)")
+    ap.add_argument("--serve", nargs="?", const="dulisun", default=None, choices=["dulisun", "zafopel"],
+                    help="instead of the RLHF iteration: prefill and decode throughput of a served family beside the one closest to it at equal "
+                    "size (dulisun: Llama, zafopel: Dulisun), with every kernel's distance from its roofline (one GPU)")
     args = ap.parse_args()
     # Libraries (NCCL's version banner, for one) write to file descriptor 1. The contract is ONE JSON line on
     # stdout, so everything else is sent to stderr and the line goes to the saved descriptor at the end.
@@ -239,10 +240,10 @@ def main() -> None:
         os.write(real_stdout, (json.dumps(obj) + "\n").encode())
 
     if args.serve:
-        from rpeg_b200.engine import serve_bench
+        from rpeg_b200.engine import serve_bench, serve_bench_latent
         sampler = ClockSampler(0)
         sampler.start()
-        line = serve_bench.run(["2b", "7b"], 4)
+        line = (serve_bench if args.serve == "dulisun" else serve_bench_latent).run(["2b", "7b"], 4)
         emit({**line, "clocks": sampler.stop()})
         return
 

@@ -454,7 +454,8 @@ class Generator:
             d = torch.tensor(dst, dtype=torch.long, device=dev)
             if len(set(self.geometry)) > 1 or self.geometry[0][1] != self.geometry[0][2]:
                 for c in (*self.kcache, *self.vcache):
-                    c[d] = c[src].unsqueeze(0)
+                    if c.numel():                        # a layer may keep no values, or nothing of its own
+                        c[d] = c[src].clone()
                 return
             pages = self.kcache[0].shape[0]              # layers of one shape: a single strided copy
             flat = self.kv_storage.view(2 * self.cfg.n_layers, pages, -1)

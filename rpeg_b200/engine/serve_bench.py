@@ -2,6 +2,8 @@
 
     python bench.py --serve                       (or: python -m rpeg_b200.engine.serve_bench --sizes 2b,7b --layers 4)
 
+``bench.py --serve zafopel`` (``engine/serve_bench_latent.py``) does the same for the Zafopel family beside this one.
+
 Both models get the same width, heads, KV heads, head size and vocabulary; the Llama feed-forward is as wide as makes its
 parameters equal to those a Dulisun token uses (chosen experts plus the shared one). Random weights, ``--layers`` layers of
 the real size (a layer's rate does not depend on how many there are). Reported per size:

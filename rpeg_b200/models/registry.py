@@ -137,9 +137,9 @@ def _latent_mixer(kind: str, m: Mapping[str, Any], where: str, index: int, befor
     if second and not 1 <= q_rank <= 8192:
         raise RuntimeConfigError(f"{where}: q_rank must lie in 1 to 8192, got {q_rank}")
     mask = m.get("mask") or {}
-    window = 0 if second else int(mask.get("size", 0))
-    if not second and window < 1:
-        raise RuntimeConfigError(f"{where}: mask.size must be at least 1")
+    window = int(mask.get("size", 0))
+    if mask and (second or window < 1):
+        raise RuntimeConfigError(f"{where}: " + ("this mixer is causal and takes no mask" if second else "mask.size must be at least 1"))
     src = m.get("kv_from")
     out = LatentMixer(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=rank, scale=float(m["scale"]), rot_base=float(rot["base"]),
                       q_rank=q_rank, window=window, sink=second, kv_from=None if src is None else int(src))

@@ -468,9 +468,12 @@ class ZafopelModel(ServedDecoder):
 
     def _nsplit(self, m: LatentMixer, rows: int, table_pages: int) -> int:
         """Splits of a decode row's pages: the fewest page times over all waves of CTAs, where a CTA costs about four pages on
-        top of its own (pipeline fill, merge)."""
+        top of its own (pipeline fill, merge). One where the CUDA cores score the latents."""
+        per_sm = K.latent_decode_ctas_per_sm(m.rank_p, m.row_width)
+        if per_sm == 0:
+            return 1
         pages = min(table_pages, (m.window - 2) // K.KV_PAGE + 2) if m.window else table_pages
-        ctas, slots = rows * -(-m.heads // 32), self._num_sms * K.latent_decode_ctas_per_sm(m.rank_p, m.row_width)
+        ctas, slots = rows * -(-m.heads // 32), self._num_sms * per_sm
         return min(range(1, min(pages, 16) + 1), key=lambda n: (-(-ctas * n // slots) * (-(-pages // n) + 4), n))
 
     def _split_buffer(self, rows: int, table_pages: int) -> torch.Tensor:
