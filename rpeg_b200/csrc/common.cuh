@@ -43,6 +43,21 @@ __device__ __forceinline__ void record_error(int* status, int code, int where, i
   }
 }
 
+// One lane of a converged warp (the same one every time). An issuing warp that runs its loops with all lanes and only predicates the issue
+// itself keeps descriptors and addresses in uniform registers; inside a branch of one lane every operand is moved there first, which
+// bounds the issue rate of small tcgen05.mma shapes.
+__device__ __forceinline__ bool elect_one() {
+  uint32_t pred = 0;
+  asm volatile(
+      "{\n\t.reg .pred p;\n\t"
+      "elect.sync _|p, 0xffffffff;\n\t"
+      "@p mov.s32 %0, 1;\n\t}"
+      : "+r"(pred));
+  return pred != 0;
+}
+// The warp's number, known to be the same in all its lanes.
+__device__ __forceinline__ int uniform_warp() { return __shfl_sync(0xffffffffu, static_cast<int>(threadIdx.x >> 5), 0); }
+
 // ---------------------------------------------------------------- mbarrier
 __device__ __forceinline__ void mbar_init(uint64_t* bar, uint32_t count) {
   asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(bar)), "r"(count) : "memory");
@@ -62,6 +77,18 @@ __device__ __forceinline__ bool mbar_try_wait(uint64_t* bar, uint32_t parity) {
   asm volatile(
       "{\n\t.reg .pred p;\n\t"
       "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
+      "selp.u32 %0, 1, 0, p;\n\t}"
+      : "=r"(ok)
+      : "r"(smem_u32(bar)), "r"(parity)
+      : "memory");
+  return ok != 0;
+}
+// Whether the phase is complete, without suspending the thread.
+__device__ __forceinline__ bool mbar_test_wait(uint64_t* bar, uint32_t parity) {
+  uint32_t ok;
+  asm volatile(
+      "{\n\t.reg .pred p;\n\t"
+      "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
       "selp.u32 %0, 1, 0, p;\n\t}"
       : "=r"(ok)
       : "r"(smem_u32(bar)), "r"(parity)
@@ -275,6 +302,10 @@ __device__ __forceinline__ uint64_t make_smem_desc_sw128(uint32_t saddr, uint32_
   d |= static_cast<uint64_t>(2) << 61;  // SWIZZLE_128B
   return d;
 }
+
+// The same descriptor `bytes` further on (the address field counts 16-byte units; shared memory ends before it wraps): one addition
+// where an issuing thread would otherwise assemble 64 bits per operand.
+__device__ __forceinline__ uint64_t smem_desc_at(uint64_t desc, uint32_t bytes) { return desc + (bytes >> 4); }
 
 // Instruction descriptor, kind::f16, bf16 x bf16 -> fp32.
 __host__ __device__ constexpr uint32_t make_idesc_bf16(int M, int N, int a_mn_major, int b_mn_major) {

@@ -18,29 +18,28 @@ struct HeadGemmCfg {
   static constexpr int A_BYTES = HG_BM * HG_BK * 2;
   static constexpr int B_BYTES = BN * HG_BK * 2;
   static constexpr int STAGE_BYTES = A_BYTES + B_BYTES;
-  static constexpr int STAGES = 4;
-  static constexpr int SMEM_BYTES = STAGES * STAGE_BYTES + 1024 + 256;
+  static constexpr int MAX_STAGES = BN == 64 ? 8 : 6;     // as many as K has blocks, up to this: short ones leave room for more CTAs per SM
+  static constexpr int smem_bytes(int stages) { return stages * STAGE_BYTES + 1024 + 256; }
 };
 
 template <int BN, bool B_KN>
 __global__ void __launch_bounds__(HG_THREADS)
 head_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ CUtensorMap tmap_b, __nv_bfloat16* __restrict__ C, int M,
-                 int N, int K, int ldc, int hsc, int a_rows, int* status) {
+                 int N, int K, int ldc, int hsc, int a_rows, int stages, int* status) {
   using Cfg = HeadGemmCfg<BN>;
-  constexpr int STAGES = Cfg::STAGES;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  uint64_t* full_bar = reinterpret_cast<uint64_t*>(smem + STAGES * Cfg::STAGE_BYTES);
-  uint64_t* empty_bar = full_bar + STAGES;
-  uint64_t* done_bar = empty_bar + STAGES;
+  uint64_t* full_bar = reinterpret_cast<uint64_t*>(smem + stages * Cfg::STAGE_BYTES);
+  uint64_t* empty_bar = full_bar + stages;
+  uint64_t* done_bar = empty_bar + stages;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(done_bar + 1);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = uniform_warp(), lane = threadIdx.x & 31;
   const int n_tiles = (N + BN - 1) / BN;
   const int n0 = (blockIdx.x % n_tiles) * BN, m0 = (blockIdx.x / n_tiles) * HG_BM, h = blockIdx.y;
   const int num_kb = (K + HG_BK - 1) / HG_BK;
   if (threadIdx.x == 0) {
-    for (int s = 0; s < STAGES; ++s) { mbar_init(&full_bar[s], 1); mbar_init(&empty_bar[s], 1); }
+    for (int s = 0; s < stages; ++s) { mbar_init(&full_bar[s], 1); mbar_init(&empty_bar[s], 1); }
     mbar_init(done_bar, 1);
     *abort_flag = 0;
     fence_mbar_init();
@@ -66,36 +65,36 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
           tma_load_3d(sb, &tmap_b, &full_bar[st], kb * HG_BK, n0, h);
         }
       };
-      const int pre = num_kb < STAGES ? num_kb : STAGES;
+      const int pre = stages;
       for (int kb = 0; kb < pre; ++kb) load_b(kb, kb);         // weights do not depend on the kernel before
       griddep_wait();
       for (int kb = 0; kb < num_kb; ++kb) {
-        const int st = kb % STAGES;
+        const int st = kb % stages;
         if (kb >= pre) {
-          if (!mbar_wait(&empty_bar[st], (static_cast<uint32_t>(kb / STAGES) & 1u) ^ 1u, abort_flag, status, 1000)) break;
+          if (!mbar_wait(&empty_bar[st], (static_cast<uint32_t>(kb / stages) & 1u) ^ 1u, abort_flag, status, 1000)) break;
           load_b(kb, st);
         }
         tma_load_3d(smem + st * Cfg::STAGE_BYTES, &tmap_a, &full_bar[st], kb * HG_BK, h, m0);
       }
     }
   } else if (warp == 1) {
-    if (lane == 0) {
-      constexpr uint32_t idesc = make_idesc_bf16(HG_BM, BN, 0, B_KN ? 1 : 0);
-      bool ok = true;
-      for (int kb = 0; kb < num_kb; ++kb) {
-        const int st = kb % STAGES;
-        if (!mbar_wait(&full_bar[st], static_cast<uint32_t>(kb / STAGES) & 1u, abort_flag, status, 1010)) { ok = false; break; }
-        tc_fence_after_sync();
-        const uint32_t sa = smem_u32(smem + st * Cfg::STAGE_BYTES), sb = sa + Cfg::A_BYTES;
+    const bool leader = elect_one();               // all lanes run the loop, one issues
+    constexpr uint32_t idesc = make_idesc_bf16(HG_BM, BN, 0, B_KN ? 1 : 0);
+    bool ok = true;
+    for (int kb = 0; kb < num_kb; ++kb) {
+      const int st = kb % stages;
+      if (!__all_sync(0xffffffffu, mbar_wait(&full_bar[st], static_cast<uint32_t>(kb / stages) & 1u, abort_flag, status, 1010))) { ok = false; break; }
+      tc_fence_after_sync();
+      const uint32_t sa = smem_u32(smem + st * Cfg::STAGE_BYTES), sb = sa + Cfg::A_BYTES;
 #pragma unroll
-        for (int k = 0; k < HG_BK / 16; ++k)
+      for (int k = 0; k < HG_BK / 16; ++k)
+        if (leader)
           umma_bf16_ss(tmem, make_smem_desc_sw128(sa + k * 32, 16, 1024),
                        B_KN ? make_smem_desc_sw128(sb + k * 2048, 64 * HG_BK * 2, 1024) : make_smem_desc_sw128(sb + k * 32, 16, 1024), idesc,
                        (kb | k) != 0 ? 1u : 0u);
-        umma_commit(&empty_bar[st]);
-      }
-      if (ok) umma_commit(done_bar);
+      if (leader) umma_commit(&empty_bar[st]);
     }
+    if (ok && leader) umma_commit(done_bar);
   } else {
     const int quad = warp & 3, r = m0 + quad * 32 + lane;
     if (__all_sync(0xffffffffu, mbar_wait(done_bar, 0, abort_flag, status, 1020)) && m0 + quad * 32 < M) {
@@ -144,13 +143,14 @@ static int launch_head_gemm(const CUtensorMap& ta, const CUtensorMap& tb, void* 
   using Cfg = HeadGemmCfg<BN>;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES) != cudaSuccess) return -20;
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::smem_bytes(Cfg::MAX_STAGES)) != cudaSuccess) return -20;
     configured = true;
   }
   const long long tiles = static_cast<long long>((N + BN - 1) / BN) * ((M + HG_BM - 1) / HG_BM);
   if (tiles > 0x7fffffffll) return -2;
-  return launch_pdl(kern, dim3(static_cast<unsigned>(tiles), H), dim3(HG_THREADS), static_cast<size_t>(Cfg::SMEM_BYTES), stream, ta, tb,
-                    static_cast<__nv_bfloat16*>(C), M, N, K, ldc, hsc, a_rows, status) == cudaSuccess ? 0 : -21;
+  const int num_kb = (K + HG_BK - 1) / HG_BK, stages = num_kb < Cfg::MAX_STAGES ? num_kb : Cfg::MAX_STAGES;
+  return launch_pdl(kern, dim3(static_cast<unsigned>(tiles), H), dim3(HG_THREADS), static_cast<size_t>(Cfg::smem_bytes(stages)), stream, ta, tb,
+                    static_cast<__nv_bfloat16*>(C), M, N, K, ldc, hsc, a_rows, stages, status) == cudaSuccess ? 0 : -21;
 }
 
 }  // namespace rpeg

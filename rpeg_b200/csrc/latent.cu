@@ -9,7 +9,8 @@
 //
 //   latent_rows        one launch between the projections and the attention: weight-scaled RMS norm of up to two segments of a
 //                      projection (a query latent to a buffer, the key/value latent to the cache), interleaved rotation of the shared
-//                      key part (to the cache) and of the queries' rotated parts
+//                      key part (to the cache) and of the queries' rotated parts, and the activation of a feed-forward whose first
+//                      product is part of the same projection
 //   latent_gather      the cache rows a prompt sees, as one contiguous matrix (the operand of the products that give its keys and values)
 //   latent_attn_rows   attention of single query rows over the cache on the CUDA cores, for fp32 and for sizes the tensor-core
 //                      kernels (latent_decode.cu, latent_prefill.cu) do not take
@@ -19,7 +20,6 @@
 namespace rpeg {
 
 constexpr int LPAGE = RPEG_KV_PAGE;
-constexpr int LR_THREADS = 128;
 
 // A projection's output: an activation [rows, ld], or `splits` fp32 partials of it.
 struct Projection {
@@ -61,6 +61,9 @@ struct LatentRows {
   int q_col0, H, dim_p;
   void* q_nope; int ld_nope;
   void* q_rot; int ld_rot, hs_rot;
+  // feed-forward: squared relu of src columns [ff_col0, + ff_p) -> ff_out [rows, ff_p]; ff_p = 0: none
+  int ff_col0, ff_p;
+  void* ff_out;
 };
 
 __device__ __forceinline__ float4 rotate_pairs(float4 u, const LatentRows& a, int p, int c) {
@@ -72,14 +75,14 @@ __device__ __forceinline__ float4 rotate_pairs(float4 u, const LatentRows& a, in
   return make_float4(u.x * s0.x - u.y * s0.y, u.y * s0.x + u.x * s0.y, u.z * s1.x - u.w * s1.y, u.w * s1.x + u.z * s1.y);
 }
 
-// The first blocks normalise (one per token and segment), the others rotate and move queries (four columns per thread).
+// The first blocks normalise (one per token and segment), the others do what is elementwise (four columns per thread).
 template <typename T, bool PARTIALS>
-__global__ void __launch_bounds__(LR_THREADS)
+__global__ void __launch_bounds__(512)
 latent_rows_kernel(const LatentRows a, int norm_blocks, int items) {
   griddep_launch();
   griddep_wait();
   extern __shared__ float rowbuf[];
-  __shared__ float part[LR_THREADS / 32];
+  __shared__ float part[16];
   if (static_cast<int>(blockIdx.x) < norm_blocks) {
     const int nseg = (a.nq > 0) + (a.rank > 0);
     const int t = blockIdx.x / nseg;
@@ -96,28 +99,28 @@ latent_rows_kernel(const LatentRows a, int norm_blocks, int items) {
       out = static_cast<T*>(a.nq_out) + static_cast<size_t>(t) * a.nq_p;
     }
     float ss = 0.f;
-    for (int c = threadIdx.x * 4; c < np; c += LR_THREADS * 4) {
+    const int all = np + (kv ? a.rot_p : 0), step = blockDim.x * 4;
+    for (int c = threadIdx.x * 4; c < all; c += step) {
       const float4 v = read_projection<T, PARTIALS>(a.src, t, col0 + c);
-      store4(rowbuf + c, v);
-      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      if (c < np) {
+        store4(rowbuf + c, v);
+        ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      } else {
+        store4(out + c, rotate_pairs(v, a, p, c - np));
+      }
     }
-    if (kv)
-      for (int c = threadIdx.x * 4; c < a.rot_p; c += LR_THREADS * 4)
-        store4(out + a.rank_p + c, rotate_pairs(read_projection<T, PARTIALS>(a.src, t, col0 + a.rank_p + c), a, p, c));
     ss = warp_sum(ss);
     if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = ss;
     __syncthreads();
-    ss = 0.f;
-#pragma unroll
-    for (int i = 0; i < LR_THREADS / 32; ++i) ss += part[i];
+    ss = warp_sum((threadIdx.x & 31) < (blockDim.x >> 5) ? part[threadIdx.x & 31] : 0.f);
     const float r = rsqrtf(ss / static_cast<float>(n) + a.eps);
-    for (int c = threadIdx.x * 4; c < np; c += LR_THREADS * 4) {      // a thread reads back only what it wrote
+    for (int c = threadIdx.x * 4; c < np; c += step) {                // a thread reads back only what it wrote
       const float4 v = load4(rowbuf + c), g = load4(w + c);
       store4(out + c, make_float4(v.x * r * g.x, v.y * r * g.y, v.z * r * g.z, v.w * r * g.w));
     }
     return;
   }
-  const long long item = static_cast<long long>(blockIdx.x - norm_blocks) * LR_THREADS + threadIdx.x;
+  const long long item = static_cast<long long>(blockIdx.x - norm_blocks) * blockDim.x + threadIdx.x;
   const int t = static_cast<int>(item / items);
   if (t >= a.rows) return;
   const int e = static_cast<int>(item - static_cast<long long>(t) * items);
@@ -126,11 +129,19 @@ latent_rows_kernel(const LatentRows a, int norm_blocks, int items) {
     const int h = e / nr, c = (e - h * nr) * 4;
     const float4 v = rotate_pairs(read_projection<T, PARTIALS>(a.src, t, a.q_col0 + h * hw + a.dim_p + c), a, a.pos[t], c);
     store4(static_cast<T*>(a.q_rot) + static_cast<size_t>(t) * a.ld_rot + h * a.hs_rot + c, v);
-  } else {
-    const int nd = a.dim_p >> 2, f = e - rot_items, h = f / nd, c = (f - h * nd) * 4;
+    return;
+  }
+  const int nd = a.dim_p >> 2, nope_items = a.q_nope != nullptr ? a.H * nd : 0;
+  if (e < rot_items + nope_items) {
+    const int f = e - rot_items, h = f / nd, c = (f - h * nd) * 4;
     store4(static_cast<T*>(a.q_nope) + static_cast<size_t>(t) * a.ld_nope + h * a.dim_p + c,
            read_projection<T, PARTIALS>(a.src, t, a.q_col0 + h * hw + c));
+    return;
   }
+  const int c = (e - rot_items - nope_items) * 4;
+  const float4 v = read_projection<T, PARTIALS>(a.src, t, a.ff_col0 + c);
+  store4(static_cast<T*>(a.ff_out) + static_cast<size_t>(t) * a.ff_p + c,
+         make_float4(ff_act<FF_RELU2>(v.x), ff_act<FF_RELU2>(v.y), ff_act<FF_RELU2>(v.z), ff_act<FF_RELU2>(v.w)));
 }
 
 // One warp per visible row: row r of request b (off[b] <= r < off[b + 1]) is position lo[b] + r - off[b] of page-table row slot[cu[b]].
@@ -148,7 +159,15 @@ latent_gather_kernel(const uint4* __restrict__ cache, int vecs, const int* __res
   const int page = page_table[static_cast<size_t>(slot[cu[b]]) * max_pages + p / LPAGE];
   const uint4* src = cache + (static_cast<size_t>(page) * LPAGE + p % LPAGE) * vecs;
   uint4* dst = out + static_cast<size_t>(r) * vecs;
-  for (int i = lane; i < vecs; i += 32) dst[i] = src[i];
+  for (int i0 = lane; i0 < vecs; i0 += 96) {                          // three loads in flight per lane
+    uint4 v[3];
+#pragma unroll
+    for (int k = 0; k < 3; ++k)
+      if (i0 + 32 * k < vecs) v[k] = src[i0 + 32 * k];
+#pragma unroll
+    for (int k = 0; k < 3; ++k)
+      if (i0 + 32 * k < vecs) dst[i0 + 32 * k] = v[k];
+  }
 }
 
 // ---------------------------------------------------------------------------------- attention on the CUDA cores
@@ -288,23 +307,28 @@ extern "C" int rpeg_latent_rows(const void* src, int splits, long long stride, i
                                 const float* cos_t, const float* sin_t, int rot, int rot_p, float eps, int nq_col0, int nq, int nq_p,
                                 const void* nq_w, void* nq_out, int kv_col0, int rank, int rank_p, const void* kv_w, void* cache,
                                 const int* page_table, int max_pages, int q_col0, int H, int dim_p, void* q_nope, int ld_nope, void* q_rot,
-                                int ld_rot, int hs_rot, int f32, void* stream) {
+                                int ld_rot, int hs_rot, int ff_col0, int ff_p, void* ff_out, int f32, void* stream) {
   if (rows <= 0) return 0;
+  if ((ff_p & 7) || (ff_col0 & 3) || ff_p < 0 || (ff_p > 0 && ff_out == nullptr)) return -2;
   if ((rot_p | nq_p | rank_p | dim_p | ld_nope | ld_rot | hs_rot) & 7 || ((ld | nq_col0 | kv_col0 | q_col0) & 3)) return -2;
   if (rot < 0 || rot > rot_p || (rot & 1) || nq > nq_p || rank > rank_p || H < 0) return -2;
   if ((nq > 0 && (nq_w == nullptr || nq_out == nullptr)) || (rank > 0 && (kv_w == nullptr || cache == nullptr || page_table == nullptr)) ||
       (H > 0 && rot_p > 0 && q_rot == nullptr))
     return -3;
   const LatentRows a{{src, splits, stride, ld}, rows, pos, slot, cos_t, sin_t, rot, rot_p, eps, nq_col0, nq, nq_p, nq_w, nq_out, kv_col0, rank,
-                     rank_p, kv_w, cache, page_table, max_pages, q_col0, H, dim_p, q_nope, ld_nope, q_rot, ld_rot, hs_rot};
+                     rank_p, kv_w, cache, page_table, max_pages, q_col0, H, dim_p, q_nope, ld_nope, q_rot, ld_rot, hs_rot, ff_col0, ff_p, ff_out};
   const long long norm_blocks = static_cast<long long>(rows) * ((nq > 0) + (rank > 0));
-  const int items = H * ((rot_p >> 2) + (q_nope != nullptr ? dim_p >> 2 : 0));
-  const long long blocks = norm_blocks + (static_cast<long long>(rows) * items + LR_THREADS - 1) / LR_THREADS;
+  const int items = H * ((rot_p >> 2) + (q_nope != nullptr ? dim_p >> 2 : 0)) + (ff_p >> 2);
+  // few tokens: a normalised row in one step of its block (its latency is all that counts); many: small blocks
+  const int widest = norm_blocks && rows <= 1024 ? (nq_p > rank_p + rot_p ? nq_p : rank_p + rot_p) : 0;
+  int threads = 128;
+  while (threads < 512 && threads * 4 < widest) threads *= 2;
+  const long long blocks = norm_blocks + (static_cast<long long>(rows) * items + threads - 1) / threads;
   if (blocks <= 0) return 0;
   const size_t smem = static_cast<size_t>(norm_blocks ? (nq_p > rank_p ? nq_p : rank_p) : 0) * 4;
   if (blocks > 0x7fffffffll || smem > 48 * 1024) return -2;
 #define RPEG_LR(T_, P_)                                                                                                                      \
-  return launch_pdl(latent_rows_kernel<T_, P_>, dim3(static_cast<unsigned>(blocks)), dim3(LR_THREADS), smem, STREAM(stream), a,              \
+  return launch_pdl(latent_rows_kernel<T_, P_>, dim3(static_cast<unsigned>(blocks)), dim3(threads), smem, STREAM(stream), a,                 \
                     static_cast<int>(norm_blocks), items) == cudaSuccess ? 0 : -21;
   if (f32) { RPEG_LR(float, false) }
   if (splits > 0) { RPEG_LR(__nv_bfloat16, true) }

@@ -1,20 +1,21 @@
 // Latent attention of single query rows on the tensor cores (bf16): up to 32 heads of one row against the cached rows themselves.
 //
-//   S[head, key]  = q_h . row_key              q_h [W] = (query through the key map | rotated part), row [W] = (latent | rotated part)
-//   P             = softmax(S * scale  [visible keys], sink)
-//   O^T[d, head]  = sum_key row_key[d] P[head, key]       for the latent's dimensions d < rank
+//   S^T[key, head]  = row_key . q_h            q_h [W] = (query through the key map | rotated part), row [W] = (latent | rotated part)
+//   P^T             = softmax over the keys (S^T * scale  [visible keys], sink)
+//   O^T[d, head]    = sum_key row_key[d] P^T[key, head]      for the latent's dimensions d < rank
 //
 // A cached row is read from memory once, for the scores of all heads and for their averages: the tile of 64 keys (one cache page) that
-// TMA brings to shared memory is the K-major operand B of the first product and, read along its other axis, the MN-major operand A
-// of the second. Roles: a TMA warp, an MMA warp, four warps of which one turns scores into weights (its lanes are the heads) while all
-// four rescale and store the accumulator (their lanes are latent dimensions).
-//   * Operand A of the first product is 128 rows high and holds 32 heads; the rows below read whatever lies there, and what they give is
-//     in TMEM lanes nobody reads.
-//   * A weight goes to the tensor cores as the sum of two bf16 numbers (16 bits), so that rounding the operands does not show: rows 0..31
-//     of the 64-row operand P are the leading parts, rows 32..63 the remainders, and the two halves of the accumulator are added in the
-//     end. Both parts cost one pass.
+// TMA brings to shared memory is operand A of both products, K-major in the first (64 x W), MN-major along its other axis in the second
+// (128 latent dimensions x 64 keys at a time). Roles: a TMA warp, an MMA warp, four warps that turn scores into weights and later
+// rescale and store the accumulator.
+//   * The 64-row scores lie in the first 16 TMEM lanes of each warp's quadrant: a warp sees 16 keys of all 32 heads. The heads are
+//     dealt to the two half warps, so a lane works on one key and 16 heads.
+//   * A weight goes to the tensor cores as the sum of two bf16 numbers (16 bits), so that rounding the operands does not show: columns
+//     0..31 of operand P are the leading parts, 32..63 the remainders, and the two halves of the accumulator are added in the end.
+//     Both parts cost one pass.
+//   * The maximum a head's weights refer to is set by the first tile and changed (and the accumulator rescaled) only when some score
+//     exceeds it by more than 8 (log2); a barrier that also takes the vote is all the warps exchange otherwise.
 //   * Scores are double buffered in TMEM, weights in shared memory: the product for the next page runs under the softmax of this one.
-//   * The accumulator is rescaled only when some head's maximum grew by more than 8 (log2).
 // Splits of a row's pages leave unnormalised partial sums; latent_merge adds them up.
 #include "act_io.cuh"
 #include "rpeg_kernels.h"
@@ -24,7 +25,7 @@ namespace rpeg {
 constexpr int LD_PAGE = RPEG_KV_PAGE, LD_HEADS = 32, LD_THREADS = 192;
 constexpr int LD_ATOM = LD_PAGE * 128;             // 64 keys x 64 columns, 128-byte swizzled
 constexpr int LD_Q_ATOM = LD_HEADS * 128;
-constexpr int LD_P_BYTES = 2 * LD_HEADS * 128;     // [leading parts; remainders] x 64 keys
+constexpr int LD_P_BYTES = LD_PAGE * 128;          // 64 keys x [leading parts; remainders] of 32 heads
 constexpr int LD_MAX_ATOMS = 9, LD_MAX_BLOCKS = 4; // rows of up to 576 elements, latents of up to 512
 constexpr float LD_RESCALE = 8.0f;
 
@@ -35,18 +36,48 @@ struct LatentDecode {
   __nv_bfloat16* out;                              // [rows, H, rank_p]
   float* partial;                                  // [rows, H, nsplit, rank_p], then (max, sum) [rows, H, nsplit]
   long long ml_offset;
-  int H, rank_p, ksteps, atoms, stage_atoms, blocks, window, nsplit, stages, tmem_cols;
+  int H, rank_p, atoms, stage_atoms, blocks, window, nsplit, stages, tmem_cols;
   float scale_log2;
   int* status;
 };
 
-__device__ __forceinline__ void bar_sync_softmax() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+// Barrier of the four softmax warps; returns whether any of their threads votes yes.
+__device__ __forceinline__ bool softmax_vote(bool yes) {
+  uint32_t any;
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\t"
+      "setp.ne.u32 q, %1, 0;\n\t"
+      "barrier.cta.red.or.pred p, 1, 128, q;\n\t"
+      "selp.u32 %0, 1, 0, p;\n\t}"
+      : "=r"(any)
+      : "r"(yes ? 1u : 0u)
+      : "memory");
+  return any != 0;
+}
+__device__ __forceinline__ void softmax_sync() { asm volatile("barrier.cta.sync 1, 128;" ::: "memory"); }
+
+// v[i] of 16 lanes -> in lane c of the 16: the maximum (or sum) of their v[c].
+template <bool MAX>
+__device__ __forceinline__ float half_warp_transpose(float (&v)[16], int lane) {
+#pragma unroll
+  for (int n = 8; n >= 1; n >>= 1) {
+    const bool up = lane & n;
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+      if (i < n) {
+        const float send = up ? v[i] : v[i + n], keep = up ? v[i + n] : v[i];
+        const float got = __shfl_xor_sync(0xffffffffu, send, n);
+        v[i] = MAX ? fmaxf(keep, got) : keep + got;
+      }
+  }
+  return v[0];
+}
 
 __global__ void __launch_bounds__(LD_THREADS, 2)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_c, const LatentDecode a) {
   extern __shared__ uint8_t smem_raw[];
-  __shared__ float alpha_sm[2][LD_HEADS], fac_sm[LD_HEADS];
-  __shared__ int flag_sm[2];
+  __shared__ float warp_part[4][LD_HEADS], alpha_sm[LD_HEADS];
+  __shared__ int failed[4];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int stage_bytes = a.stage_atoms * LD_ATOM;
   uint8_t* q_sm = smem;
@@ -64,10 +95,12 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
 
   const int row = blockIdx.x, h0 = blockIdx.y * LD_HEADS, split = blockIdx.z;
   const int nh = min(LD_HEADS, a.H - h0);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = uniform_warp(), lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
+    tma_prefetch_desc(&tmap_q);
+    tma_prefetch_desc(&tmap_c);
     mbar_init(q_full, 1);
-    for (int i = 0; i < 2; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_full[i], 1); mbar_init(&pv_done[i], 1); }
+    for (int i = 0; i < 2; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_full[i], 4); mbar_init(&pv_done[i], 1); }
     for (int s = 0; s < a.stages; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
     *abort_flag = 0;
     fence_mbar_init();
@@ -86,173 +119,231 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
   const int key0 = a.window > 0 ? max(0, L - a.window) : 0;
   const int pg0 = key0 / LD_PAGE, pg1 = L > 0 ? (L + LD_PAGE - 1) / LD_PAGE : pg0;
   const int per = (pg1 - pg0 + a.nsplit - 1) / a.nsplit;
-  const int pa = min(pg1, pg0 + split * per), n_tiles = min(pg1, pa + per) - pa;
+  const int pa = min(pg1, pg0 + split * per);
+  const int n_tiles = __shfl_sync(0xffffffffu, min(pg1, pa + per) - pa, 0);
+  auto parity2 = [](int j) { return static_cast<uint32_t>(j >> 1) & 1u; };      // of the phase tile j completes on a pair of barriers
+  constexpr int O_COL = 2 * LD_HEADS;                                            // TMEM: two score buffers, then the accumulator
 
   if (warp == 0) {
     if (lane == 0 && n_tiles > 0) {
       const int* pt = a.page_table + static_cast<size_t>(a.slot[row]) * a.max_pages;
       mbar_expect_tx(q_full, a.atoms * LD_Q_ATOM);
       for (int c = 0; c < a.atoms; ++c) tma_load_2d(q_sm + c * LD_Q_ATOM, &tmap_q, q_full, c * 64, row * a.H + h0);
+      int st = 0;
+      uint32_t phase = 1u;
+      int page = pt[pa];
       for (int j = 0; j < n_tiles; ++j) {
-        const int st = j % a.stages;
-        if (!mbar_wait(&empty[st], (static_cast<uint32_t>(j / a.stages) & 1u) ^ 1u, abort_flag, a.status, 1100)) break;
+        const int y = page * LD_PAGE;
+        if (j + 1 < n_tiles) page = pt[pa + j + 1];              // the next page's number arrives under this page's copies
+        if (!mbar_wait(&empty[st], phase, abort_flag, a.status, 1100)) break;
         mbar_expect_tx(&full[st], a.atoms * LD_ATOM);
-        const int y = pt[pa + j] * LD_PAGE;
-        for (int c = 0; c < a.atoms; ++c) tma_load_2d(c_sm + st * stage_bytes + c * LD_ATOM, &tmap_c, &full[st], c * 64, y);
+        uint8_t* dst = c_sm + st * stage_bytes;
+        for (int c = 0; c < a.atoms; ++c) tma_load_2d(dst + c * LD_ATOM, &tmap_c, &full[st], c * 64, y);
+        if (++st == a.stages) { st = 0; phase ^= 1u; }
       }
     }
   } else if (warp == 1) {
-    if (lane == 0 && n_tiles > 0) {
-      constexpr uint32_t idesc_s = make_idesc_bf16(128, LD_PAGE, 0, 0);
-      constexpr uint32_t idesc_o = make_idesc_bf16(128, 2 * LD_HEADS, 1, 0);
-      auto scores = [&](int j) -> bool {
-        const int st = j % a.stages;
-        if (!mbar_wait(&full[st], static_cast<uint32_t>(j / a.stages) & 1u, abort_flag, a.status, 1110)) return false;
+    if (n_tiles > 0) {                               // all lanes, converged; one of them issues
+      const bool leader = elect_one();
+      constexpr uint32_t idesc_s = make_idesc_bf16(LD_PAGE, LD_HEADS, 0, 0);
+      constexpr uint32_t idesc_o = make_idesc_bf16(128, 2 * LD_HEADS, 1, 1);
+      const uint64_t q_desc = make_smem_desc_sw128(smem_u32(q_sm), 16, 1024);
+      const uint64_t ck_desc = make_smem_desc_sw128(smem_u32(c_sm), 16, 1024);            // keys as rows of the first product
+      const uint64_t cv_desc = make_smem_desc_sw128(smem_u32(c_sm), LD_ATOM, 1024);       // the same keys along their other axis
+      const uint64_t p_desc = make_smem_desc_sw128(smem_u32(p_sm), LD_P_BYTES, 1024);
+      int qs = 0, ps = 0;                   // stages of the next score and the next average
+      uint32_t q_phase = 0u;
+      auto scores = [&](int j) {
         tc_fence_after_sync();
-        const uint32_t q_addr = smem_u32(q_sm), c_addr = smem_u32(c_sm + st * stage_bytes), ts = tmem + (j & 1) * LD_PAGE;
-#pragma unroll 4
-        for (int k = 0; k < a.ksteps; ++k) {
-          const uint32_t in = static_cast<uint32_t>(k & 3) * 32;
-          umma_bf16_ss(ts, make_smem_desc_sw128(q_addr + (k >> 2) * LD_Q_ATOM + in, 16, 1024),
-                       make_smem_desc_sw128(c_addr + (k >> 2) * LD_ATOM + in, 16, 1024), idesc_s, k != 0 ? 1u : 0u);
-        }
-        umma_commit(&s_full[j & 1]);
-        return true;
-      };
-      bool ok = mbar_wait(q_full, 0, abort_flag, a.status, 1111);
-      if (ok) ok = scores(0);
-      for (int j = 0; j < n_tiles && ok; ++j) {
-        if (j + 1 < n_tiles && !scores(j + 1)) break;
-        if (!mbar_wait(&p_full[j & 1], static_cast<uint32_t>(j >> 1) & 1u, abort_flag, a.status, 1112)) break;
-        tc_fence_after_sync();
-        const int st = j % a.stages;
-        const uint32_t c_addr = smem_u32(c_sm + st * stage_bytes), p_addr = smem_u32(p_sm + (j & 1) * LD_P_BYTES);
-        for (int blk = 0; blk < a.blocks; ++blk)
+        const uint32_t ts = tmem + (j & 1) * LD_HEADS;
+        uint64_t qd = q_desc, cd = smem_desc_at(ck_desc, qs * stage_bytes);
+        for (int c = 0; c < a.atoms; ++c) {                       // columns past the row's end are zeros in both operands
 #pragma unroll
-          for (int k = 0; k < LD_PAGE / 16; ++k)       // 16 keys: 16 rows (2 KiB) of every 64-column atom
-            umma_bf16_ss(tmem + 2 * LD_PAGE + blk * (2 * LD_HEADS), make_smem_desc_sw128(c_addr + 2 * blk * LD_ATOM + k * 2048, LD_ATOM, 1024),
-                         make_smem_desc_sw128(p_addr + k * 32, 16, 1024), idesc_o, (j | k) != 0 ? 1u : 0u);
-        umma_commit(&pv_done[j & 1]);
-        umma_commit(&empty[st]);
+          for (int k = 0; k < 4; ++k)
+            if (leader) umma_bf16_ss(ts, smem_desc_at(cd, k * 32), smem_desc_at(qd, k * 32), idesc_s, (c | k) != 0 ? 1u : 0u);
+          qd = smem_desc_at(qd, LD_Q_ATOM);
+          cd = smem_desc_at(cd, LD_ATOM);
+        }
+        if (leader) umma_commit(&s_full[j & 1]);
+        if (++qs == a.stages) { qs = 0; q_phase ^= 1u; }
+      };
+      auto averages = [&](int j) {
+        tc_fence_after_sync();
+        const uint64_t pd = smem_desc_at(p_desc, (j & 1) * LD_P_BYTES);
+        uint64_t cd = smem_desc_at(cv_desc, ps * stage_bytes);
+        uint32_t to = tmem + O_COL;
+        for (int blk = 0; blk < a.blocks; ++blk) {
+#pragma unroll
+          for (int k = 0; k < LD_PAGE / 16; ++k)                  // 16 keys: 16 rows (2 KiB) of both operands' atoms
+            if (leader) umma_bf16_ss(to, smem_desc_at(cd, k * 2048), smem_desc_at(pd, k * 2048), idesc_o, (j | k) != 0 ? 1u : 0u);
+          cd = smem_desc_at(cd, 2 * LD_ATOM);
+          to += 2 * LD_HEADS;
+        }
+        if (leader) {
+          umma_commit(&pv_done[j & 1]);
+          umma_commit(&empty[ps]);
+        }
+        if (++ps == a.stages) ps = 0;
+      };
+      // Whatever is ready next: averages (they free a stage), else scores of a tile that has arrived, one tile ahead of the weights at
+      // most. With two stages in flight a fixed order would make one of them wait for the other's copy.
+      auto wait = [&](uint64_t* bar, uint32_t parity, int where) -> bool {
+        return __all_sync(0xffffffffu, mbar_wait(bar, parity, abort_flag, a.status, where));
+      };
+      auto arrived = [&](uint64_t* bar, uint32_t parity) -> bool { return __all_sync(0xffffffffu, mbar_test_wait(bar, parity)); };
+      bool ok = wait(q_full, 0, 1111);
+      int jq = 0, jp = 0;
+      while (ok && jp < n_tiles) {
+        const bool can_q = jq < n_tiles && jq <= jp + 1, can_p = jp < jq;
+        if (can_q && can_p) {
+          uint64_t t0 = 0;
+          for (uint32_t spin = 1;; ++spin) {
+            if (arrived(&p_full[jp & 1], parity2(jp))) { averages(jp++); break; }
+            if (arrived(&full[qs], q_phase)) { scores(jq++); break; }
+            if ((spin & 1023u) == 0u) {
+              if (t0 == 0) t0 = global_timer_ns();
+              if (__any_sync(0xffffffffu, *abort_flag || global_timer_ns() - t0 > RPEG_WAIT_LIMIT_NS)) {
+                *abort_flag = 1;
+                if (leader) record_error(a.status, RPEG_ERR_MBAR_TIMEOUT, 1112, jp);
+                ok = false;
+                break;
+              }
+            }
+          }
+        } else if (can_q) {
+          ok = wait(&full[qs], q_phase, 1110);
+          if (ok) scores(jq++);
+        } else {
+          ok = wait(&p_full[jp & 1], parity2(jp), 1113);
+          if (ok) averages(jp++);
+        }
       }
     }
   } else {
     const int quad = warp & 3;
-    const bool leader = quad == 0;                  // this warp's TMEM lanes are the heads of S
-    const uint32_t lanes = static_cast<uint32_t>(quad * 32) << 16;
-    const uint32_t to = tmem + lanes + 2 * LD_PAGE;
-    float m_ref = -INFINITY, l = 0.f;
-    for (int n = 0; n < n_tiles; ++n) {
-      uint32_t s[2][32];
-      if (leader) {
-        int flag = 0;
-        const bool ok = __all_sync(0xffffffffu, mbar_wait(&s_full[n & 1], static_cast<uint32_t>(n >> 1) & 1u, abort_flag, a.status, 1120));
-        if (ok) {
-          tc_fence_after_sync();
-          tmem_ld_32x32(tmem + (n & 1) * LD_PAGE, s[0]);
-          tmem_ld_32x32(tmem + (n & 1) * LD_PAGE + 32, s[1]);
-          tmem_wait_ld();
-          const int k0 = (pa + n) * LD_PAGE;
-          const bool edge = k0 < key0 || k0 + LD_PAGE > L;           // uniform
-          float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+    const uint32_t lanes = tmem + (static_cast<uint32_t>(quad * 32) << 16);
+    const uint32_t to = lanes + O_COL;
+    const int key = quad * 16 + (lane & 15);         // of the tile; this lane's heads: (lane >> 4) * 16 + i
+    const float scale = a.scale_log2;
+    float m_ref = -INFINITY;                         // of head `lane`, the same in all four warps
+    float shift[16], l[16];                          // of the lane's 16 heads: what m_ref is, sum of the weights of this lane's keys
 #pragma unroll
-          for (int i = 0; i < 64; ++i) {
-            float v = __uint_as_float(s[i >> 5][i & 31]) * a.scale_log2;
-            if (edge && (k0 + i < key0 || k0 + i >= L)) v = -INFINITY;
-            s[i >> 5][i & 31] = __float_as_uint(v);
-            mx[i & 3] = fmaxf(mx[i & 3], v);
-          }
-          const float tmax = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
-          float al = 1.f;
-          if (lane < nh) {
-            if (n == 0) {
-              m_ref = tmax;
-            } else if (tmax > m_ref + LD_RESCALE) {
-              al = exp2f(m_ref - tmax);
-              m_ref = tmax;
-              l *= al;
-            }
-          }
-          alpha_sm[n & 1][lane] = al;
-          flag = __any_sync(0xffffffffu, al != 1.f) ? 1 : 0;
-        } else {
-          flag = 2;
+    for (int i = 0; i < 16; ++i) { shift[i] = 0.f; l[i] = 0.f; }
+    bool alive = true;
+    for (int n = 0; n < n_tiles && alive; ++n) {
+      const bool ok = __all_sync(0xffffffffu, mbar_wait(&s_full[n & 1], parity2(n), abort_flag, a.status, 1120));
+      float x[16];
+      {
+        uint32_t s[32];
+        tc_fence_after_sync();
+        tmem_ld_32x32(lanes + (n & 1) * LD_HEADS, s);
+        tmem_wait_ld();
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const float other = __shfl_sync(0xffffffffu, __uint_as_float(s[16 + i]), lane & 15);
+          x[i] = lane < 16 ? __uint_as_float(s[i]) : other;
         }
-        if (lane == 0) flag_sm[n & 1] = flag;
       }
-      bar_sync_softmax();
-      const int flag = flag_sm[n & 1];
-      if (flag == 2) break;
-      if (flag == 1) {
-        if (__all_sync(0xffffffffu, mbar_wait(&pv_done[(n - 1) & 1], static_cast<uint32_t>((n - 1) >> 1) & 1u, abort_flag, a.status, 1121))) {
-          tc_fence_after_sync();
+      const int k0 = (pa + n) * LD_PAGE;
+      if (k0 + key < key0 || k0 + key >= L) {
+#pragma unroll
+        for (int i = 0; i < 16; ++i) x[i] = -INFINITY;
+      }
+      float over = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < 16; ++i) over = fmaxf(over, fmaf(x[i], scale, -shift[i]));
+      if (softmax_vote(n == 0 || !ok || over > LD_RESCALE)) {
+        // rare: every head's maximum over the tile, new references, and the accumulator under them
+        if (lane == 0) failed[quad] = ok ? 0 : 1;
+        float t[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) t[i] = x[i];
+        warp_part[quad][lane] = half_warp_transpose<true>(t, lane);        // (scale > 0)
+        softmax_sync();
+        if (failed[0] | failed[1] | failed[2] | failed[3]) { alive = false; break; }
+        const float tmax = fmaxf(fmaxf(warp_part[0][lane], warp_part[1][lane]), fmaxf(warp_part[2][lane], warp_part[3][lane])) * scale;
+        float al = 1.f;
+        if (n == 0) {
+          m_ref = tmax;
+        } else if (tmax > m_ref + LD_RESCALE) {
+          al = exp2f(m_ref - tmax);
+          m_ref = tmax;
+        }
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          shift[i] = __shfl_sync(0xffffffffu, m_ref, (lane & 16) + i);
+          l[i] *= __shfl_sync(0xffffffffu, al, (lane & 16) + i);
+        }
+        if (n > 0) {
+          if (quad == 0) alpha_sm[lane] = al;
+          softmax_sync();
+          if (__all_sync(0xffffffffu, mbar_wait(&pv_done[(n - 1) & 1], parity2(n - 1), abort_flag, a.status, 1121))) {
+            tc_fence_after_sync();
 #pragma unroll 1
-          for (int c = 0; c < 2 * a.blocks; ++c) {
-            uint32_t v[32];
-            tmem_ld_32x32(to + c * 32, v);
-            tmem_wait_ld();
+            for (int c = 0; c < 2 * a.blocks; ++c) {
+              uint32_t v[32];
+              tmem_ld_32x32(to + c * 32, v);
+              tmem_wait_ld();
 #pragma unroll
-            for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * alpha_sm[n & 1][i]);
-            tmem_st_32x32(to + c * 32, v);
+              for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * alpha_sm[i]);
+              tmem_st_32x32(to + c * 32, v);
+            }
+            tmem_wait_st();
           }
-          tmem_wait_st();
         }
-        tc_fence_before_sync();
-        bar_sync_softmax();
+        softmax_sync();                               // the exchange buffers may be written again
       }
-      if (leader) {
-        // the buffer of this tile's weights is free once the tile before the last has been multiplied
-        if (n >= 2 && !__all_sync(0xffffffffu, mbar_wait(&pv_done[n & 1], static_cast<uint32_t>((n - 2) >> 1) & 1u, abort_flag, a.status, 1122))) {
-          // give the others their way out at the next tile: this one is never handed on, so no wait behind it can end well
-          continue;
-        }
-        uint8_t* prow = p_sm + (n & 1) * LD_P_BYTES + lane * 128;
-        float sum[2] = {0.f, 0.f};
+      // the buffer of this tile's weights is free once the tile before the last has been multiplied
+      if (n >= 2) mbar_wait(&pv_done[n & 1], parity2(n - 2), abort_flag, a.status, 1122);
+      uint8_t* prow = p_sm + (n & 1) * LD_P_BYTES + key * 128;
+      const int chunk0 = lane >> 4 << 1, sw = key & 7;
 #pragma unroll
-        for (int c = 0; c < 8; ++c) {
-          uint32_t head[4], rest[4];
+      for (int c = 0; c < 2; ++c) {                   // 8 heads: 16 bytes of leading parts, 16 of remainders
+        uint32_t head[4], rest[4];
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int i = c * 8 + 2 * e;
-            float p0 = exp2f(__uint_as_float(s[i >> 5][i & 31]) - m_ref), p1 = exp2f(__uint_as_float(s[i >> 5][(i & 31) + 1]) - m_ref);
-            if (lane >= nh) p0 = p1 = 0.f;
-            sum[0] += p0;
-            sum[1] += p1;
-            const uint32_t w0 = __float_as_uint(p0), w1 = __float_as_uint(p1);
-            head[e] = __byte_perm(w0, w1, 0x7632);
-            rest[e] = pack_bf16x2(p0 - __uint_as_float(w0 & 0xffff0000u), p1 - __uint_as_float(w1 & 0xffff0000u));
-          }
-          const int at = (c ^ (lane & 7)) << 4;
-          *reinterpret_cast<uint4*>(prow + at) = make_uint4(head[0], head[1], head[2], head[3]);
-          *reinterpret_cast<uint4*>(prow + LD_HEADS * 128 + at) = make_uint4(rest[0], rest[1], rest[2], rest[3]);
+        for (int e = 0; e < 4; ++e) {
+          const int i = c * 8 + 2 * e;
+          const float p0 = exp2f(fmaf(x[i], scale, -shift[i])), p1 = exp2f(fmaf(x[i + 1], scale, -shift[i + 1]));
+          l[i] += p0;
+          l[i + 1] += p1;
+          // leading part: the upper 16 bits as they are; the remainder is exact in fp32 and rounded to bf16
+          const uint32_t w0 = __float_as_uint(p0), w1 = __float_as_uint(p1);
+          head[e] = __byte_perm(w0, w1, 0x7632);
+          rest[e] = pack_bf16x2(p0 - __uint_as_float(w0 & 0xffff0000u), p1 - __uint_as_float(w1 & 0xffff0000u));
         }
-        l += sum[0] + sum[1];
-        fence_proxy_async_smem();
-        tc_fence_before_sync();
-        __syncwarp();
-        if (lane == 0) mbar_arrive(&p_full[n & 1]);
+        *reinterpret_cast<uint4*>(prow + (((chunk0 + c) ^ sw) << 4)) = make_uint4(head[0], head[1], head[2], head[3]);
+        *reinterpret_cast<uint4*>(prow + (((4 + chunk0 + c) ^ sw) << 4)) = make_uint4(rest[0], rest[1], rest[2], rest[3]);
       }
+      fence_proxy_async_smem();
+      tc_fence_before_sync();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&p_full[n & 1]);
     }
-    if (leader) {
+    // sums of all keys, and every head's factor (or what the merge needs)
+    warp_part[quad][lane] = half_warp_transpose<false>(l, lane);
+    softmax_sync();
+    if (quad == 0) {
+      const float sum = (warp_part[0][lane] + warp_part[1][lane]) + (warp_part[2][lane] + warp_part[3][lane]);
       float f = 1.f;
       if (a.nsplit == 1) {
         const float sl = a.sink != nullptr && lane < nh ? a.sink[h0 + lane] * 1.4426950408889634f : -INFINITY;
         const float nm = fmaxf(m_ref, sl);
         const float w = m_ref == -INFINITY ? 0.f : exp2f(m_ref - nm);
-        const float gl = l * w + (sl == -INFINITY ? 0.f : exp2f(sl - nm));
+        const float gl = sum * w + (sl == -INFINITY ? 0.f : exp2f(sl - nm));
         f = gl > 0.f ? w / gl : 0.f;
       } else if (lane < nh) {
         float2* ml = reinterpret_cast<float2*>(a.partial + a.ml_offset);
-        ml[(static_cast<size_t>(row) * a.H + h0 + lane) * a.nsplit + split] = make_float2(m_ref, l);
+        ml[(static_cast<size_t>(row) * a.H + h0 + lane) * a.nsplit + split] = make_float2(m_ref, sum);
       }
-      fac_sm[lane] = f;
+      alpha_sm[lane] = f;
     }
-    bar_sync_softmax();
+    softmax_sync();
     const int last = n_tiles - 1;
-    const bool have = n_tiles > 0 &&
-                      __all_sync(0xffffffffu, mbar_wait(&pv_done[last & 1], static_cast<uint32_t>(last >> 1) & 1u, abort_flag, a.status, 1123));
+    const bool have = n_tiles > 0 && __all_sync(0xffffffffu, mbar_wait(&pv_done[last & 1], parity2(last), abort_flag, a.status, 1123));
     tc_fence_after_sync();
     if (have || (n_tiles <= 0 && a.nsplit == 1)) {
+      const size_t at = static_cast<size_t>(row) * a.H + h0;
+      const size_t pitch = static_cast<size_t>(a.nsplit) * a.rank_p;           // partial sums: head to head
 #pragma unroll 1
       for (int blk = 0; blk < a.blocks; ++blk) {
         uint32_t v[32], u[32];
@@ -262,14 +353,18 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
           tmem_wait_ld();
         }
         const int d = blk * 128 + quad * 32 + lane;
-        if (d < a.rank_p) {
+        if (d >= a.rank_p) continue;
+        if (a.nsplit == 1) {
+          __nv_bfloat16* o = a.out + at * a.rank_p + d;
+#pragma unroll
+          for (int h = 0; h < LD_HEADS; ++h)
+            if (h < nh) o[h * a.rank_p] = __float2bfloat16(have ? (__uint_as_float(v[h]) + __uint_as_float(u[h])) * alpha_sm[h] : 0.f);
+        } else {
+          float* o = a.partial + at * pitch + static_cast<size_t>(split) * a.rank_p + d;
 #pragma unroll
           for (int h = 0; h < LD_HEADS; ++h) {
-            if (h >= nh) break;
-            const float o = have ? __uint_as_float(v[h]) + __uint_as_float(u[h]) : 0.f;
-            const size_t at = static_cast<size_t>(row) * a.H + h0 + h;
-            if (a.nsplit == 1) a.out[at * a.rank_p + d] = __float2bfloat16(o * fac_sm[h]);
-            else a.partial[(at * a.nsplit + split) * a.rank_p + d] = o;
+            if (h < nh) *o = __uint_as_float(v[h]) + __uint_as_float(u[h]);
+            o += pitch;
           }
         }
       }
@@ -334,7 +429,8 @@ static bool latent_shape(int rank_p, int W, LatentShape* s) {
   if (st < 2) st = (226 * 1024 - fixed) / stage;
   if (st < 2) return false;
   s->stages = st > 4 ? 4 : st;
-  s->tmem_cols = 2 * LD_PAGE + s->blocks * 2 * LD_HEADS <= 256 ? 256 : 512;
+  s->tmem_cols = 128;
+  while (s->tmem_cols < 2 * LD_HEADS + s->blocks * 2 * LD_HEADS) s->tmem_cols *= 2;
   if (s->tmem_cols == 512) s->ctas_per_sm = 1;
   s->smem = fixed + s->stages * stage;
   return true;
@@ -359,7 +455,7 @@ extern "C" int rpeg_latent_decode(const void* q, const void* cache, long long nu
                                   const int* pos, const int* lens, const float* sink, void* out, float* scratch, int rows, int H, int rank_p,
                                   int W, int window, int nsplit, float scale, int* status, void* stream) {
   if (rows <= 0) return 0;
-  if (((rank_p | W) & 7) || rank_p < 8 || W < rank_p || H < 1 || window < 0 || nsplit < 1 || nsplit > 64) return -2;
+  if (((rank_p | W) & 7) || rank_p < 8 || W < rank_p || H < 1 || window < 0 || nsplit < 1 || nsplit > 64 || !(scale > 0.f)) return -2;
   LatentShape s;
   if (!latent_shape(rank_p, W, &s)) return -3;
   if (nsplit > 1 && scratch == nullptr) return -6;
@@ -377,7 +473,7 @@ extern "C" int rpeg_latent_decode(const void* q, const void* cache, long long nu
     configured = s.smem;
   }
   const long long ml = static_cast<long long>(rows) * H * nsplit * rank_p;
-  const LatentDecode a{page_table, max_pages, slot, pos, lens, sink, static_cast<__nv_bfloat16*>(out), scratch, ml, H, rank_p, (W + 15) / 16, s.atoms,
+  const LatentDecode a{page_table, max_pages, slot, pos, lens, sink, static_cast<__nv_bfloat16*>(out), scratch, ml, H, rank_p, s.atoms,
                        s.stage_atoms, s.blocks, window, nsplit, s.stages, s.tmem_cols, scale * 1.4426950408889634f, status};
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   if (launch_pdl(latent_decode_kernel, dim3(rows, (H + LD_HEADS - 1) / LD_HEADS, nsplit), dim3(LD_THREADS), static_cast<size_t>(s.smem), st, tq, tc,

@@ -213,7 +213,8 @@ int rpeg_stream_update(int kind_a, const void* a, int splits_a, long long stride
 int rpeg_latent_rows(const void* src, int splits, long long stride, int ld, int rows, const int* pos, const int* slot, const float* cos_t,
                      const float* sin_t, int rot, int rot_p, float eps, int nq_col0, int nq, int nq_p, const void* nq_w, void* nq_out,
                      int kv_col0, int rank, int rank_p, const void* kv_w, void* cache, const int* page_table, int max_pages, int q_col0,
-                     int H, int dim_p, void* q_nope, int ld_nope, void* q_rot, int ld_rot, int hs_rot, int f32, void* stream);
+                     int H, int dim_p, void* q_nope, int ld_nope, void* q_rot, int ld_rot, int hs_rot, int ff_col0, int ff_p, void* ff_out, int f32,
+                     void* stream);
 int rpeg_latent_gather(const void* cache, int row_bytes, const int* page_table, int max_pages, const int* slot, const int* cu, const int* off,
                        const int* lo, int B, int rows, void* out, void* stream);
 int rpeg_latent_attn_rows(const void* q, const void* cache, const int* page_table, int max_pages, const int* slot, const int* pos,

@@ -180,9 +180,14 @@ def decode_kernels(tab: S.Table, z, d, ll, B: int, ctx: int) -> None:
     ys = K.MoEOutput(K.moe_gemm(act[0], p[0]["w_down"], rt[0][4], e.experts, 0), rt[0][4].row_of, None, 0)
     tab.add(ph, "z stream update + expert sum + norm", [lambda: K.stream_update(po, ys, z.alpha[0], p[0]["norm1"], p[0]["norm1.b"], x32) for _ in L],
             B * w * (4.0 * po.splits + 2.0 * e.top + 10), like="expert sum + norm + fp32 residual")
+    # a layer with a dense feed-forward of the chosen experts' size: its first product rides on the input projection
     ff = e.ff * e.top
-    wu = [torch.randn(ff, w, **bf) for _ in range(4)]
-    tab.add(ph, "z dense up gemm + relu2", [lambda i=i: K.ff_first(h, wu[i], "relu2") for i in C], 2.0 * ff * w, like="experts up gemm + gelu")
+    wu = [torch.randn(m.q_in + m.kv_in + ff, w, **bf) for _ in range(4)]
+    tab.add(ph, "z input projection + dense up gemm (split-K)", [lambda i=i: K.gemm_partials(h, wu[i], ws) for i in C], 2.0 * wu[0].numel(), like="llama gate/up gemm (split-K)")
+    pd, fa = K.gemm_partials(h, wu[0], ws), torch.empty(B, ff, **bf)
+    tab.add(ph, "z latent norms + rotation + append + relu2", [lambda i=i: K.latent_rows(pd, pos, slot, cos_t, sin_t, m.rot_dim, m.rot_p, 1e-6,
+            q_latent=(0, m.q_rank, p[0]["q_norm"], cq), kv=(m.q_in, m.kv_rank, p[0]["kv_norm"], cache[i], table), ff=(m.q_in + m.kv_in, fa)) for i in C],
+            (4.0 * pd.splits + 2) * B * (m.q_in + m.kv_in + ff), like="rotary + unit norm + append")
 
 
 def run(sizes: List[str], layers: int, kernels: bool = True) -> dict:

@@ -13,8 +13,8 @@ Every layer has its own sizes.
 What runs where:
   * stream, norms, angles, scores, softmax, routing are fp32; the matrix products take bf16 operands and accumulate in fp32
     (``dtype=torch.float32`` runs everything in true fp32);
-  * one projection per layer gives the query side, the latent and (decode) the router logits; one kernel then normalises, rotates and
-    writes the latents into the cache (``ops.kernels.latent_rows``);
+  * one projection per layer gives the query side, the latent and (decode) the router logits or a dense feed-forward's first
+    product; one kernel then normalises, rotates, takes the activation and writes the latents into the cache (``ops.kernels.latent_rows``);
   * decoded tokens and short portions never form keys or values: queries go through U_i transposed and score the cached rows, and
     the averaged latents go through V_i (``head_gemm`` before and after the attention). Longer portions gather the rows they see, form
     keys and values with one GEMM and run an ordinary tensor-core attention over them. ``_forms_keys`` picks the cheaper way;
@@ -100,6 +100,10 @@ class DenseFF:
     def ff_p(self) -> int:
         return pad8(self.ff)
 
+    @property
+    def in_p(self) -> int:
+        return self.ff_p
+
 
 @dataclass(frozen=True)
 class InputScaledMixture:
@@ -113,7 +117,7 @@ class InputScaledMixture:
         return pad8(self.ff)
 
     @property
-    def router_p(self) -> int:
+    def in_p(self) -> int:
         return pad8(self.experts)
 
 
@@ -123,8 +127,9 @@ class ParallelLayer:
     mlp: Optional[Union[DenseFF, InputScaledMixture]] = None
 
     @property
-    def router_in(self) -> int:
-        return self.mlp.router_p if isinstance(self.mlp, InputScaledMixture) else 0
+    def ff_in(self) -> int:
+        """Rows of the layer's input projection that belong to the feed-forward: the router, or a dense one's first product."""
+        return 0 if self.mlp is None else self.mlp.in_p
 
 
 @dataclass(frozen=True)
@@ -173,7 +178,7 @@ class ZafopelLayout(FlatLayout):
             m, e = layer.mixer, layer.mlp
             self.add(f"l{i}.norm1", d)
             self.add(f"l{i}.norm1.b", d)
-            self.add(f"l{i}.w_in", m.q_in + m.kv_in + layer.router_in, d)      # queries (or their latent), latent and rotated part, router
+            self.add(f"l{i}.w_in", m.q_in + m.kv_in + layer.ff_in, d)          # queries (or their latent), latent and rotated part, router or dense up
             if m.q_rank:
                 self.add(f"l{i}.q_norm", m.q_rank_p)
                 self.add(f"l{i}.w_uq", m.q_width, m.q_rank_p)
@@ -182,7 +187,6 @@ class ZafopelLayout(FlatLayout):
             self.add(f"l{i}.w_ukv", m.heads * (m.dim_p + m.vdim_p), m.rank_p)  # key maps of all heads, then value maps
             self.add(f"l{i}.wo", d, m.heads * m.vdim_p)
             if isinstance(e, DenseFF):
-                self.add(f"l{i}.w_up", e.ff_p, d)
                 self.add(f"l{i}.w_down", d, e.ff_p)
             elif e is not None:
                 self.add(f"l{i}.w_gate_up", e.experts, 2 * e.ff_p, d)
@@ -326,12 +330,16 @@ class ZafopelModel(ServedDecoder):
 
     def put_dense(self, i: int, up: torch.Tensor, down: torch.Tensor) -> None:
         d, f = self.cfg.width, self.cfg.layers[i].mlp.ff
-        self.p[f"l{i}.w_up"][:f, :d].copy_(up)
+        self._ff_rows(i)[:f, :d].copy_(up)
         self.p[f"l{i}.w_down"][:d, :f].copy_(down)
 
     def put_router(self, i: int, w: torch.Tensor) -> None:
-        m, e = self.cfg.layers[i].mixer, self.cfg.layers[i].mlp
-        self.p[f"l{i}.w_in"][m.q_in + m.kv_in:][: e.experts, : self.cfg.width].copy_(w)
+        self._ff_rows(i)[: w.shape[0], : self.cfg.width].copy_(w)
+
+    def _ff_rows(self, i: int) -> torch.Tensor:
+        """The feed-forward's rows of the input projection."""
+        m = self.cfg.layers[i].mixer
+        return self.p[f"l{i}.w_in"][m.q_in + m.kv_in:]
 
     def put_expert(self, i: int, s: int, gate: torch.Tensor, up: torch.Tensor, down: torch.Tensor) -> None:
         d, e = self.cfg.width, self.cfg.layers[i].mlp
@@ -366,9 +374,10 @@ class ZafopelModel(ServedDecoder):
         scored = maps * sum(spans.lens) + pairs * -(-m.heads // 32) * 128 * 2 * m.row_width
         return formed <= scored
 
-    def _attention(self, i: int, h: torch.Tensor, proj, pos, slot, page_table, cache, decode: bool, form, attend) -> torch.Tensor:
+    def _attention(self, i: int, h: torch.Tensor, proj, pos, slot, page_table, cache, decode: bool, form, attend, ff=None) -> torch.Tensor:
         """Attention of layer ``i`` up to the output projection's operand ``[T, heads * vdim_p]``; ``cache`` is the cache it reads (and, if it is
-        the layer's own, appends to). ``form``: keys and values are formed (a prefill's spans), else ``attend(m, q)`` scores the latents."""
+        the layer's own, appends to). ``form``: keys and values are formed (a prefill's spans), else ``attend(m, q)`` scores the latents.
+        ``ff``: (column of ``proj``, buffer) of a dense feed-forward whose activation is taken along."""
         m, p, T, eps = self.cfg.layers[i].mixer, self.p, h.shape[0], self.cfg.norm_eps
         bf = dict(dtype=self.dtype, device=self.device)
         cos_t, sin_t = self._tables.get((m.rot_base, m.rot_dim), (None, None))
@@ -376,8 +385,8 @@ class ZafopelModel(ServedDecoder):
         src = proj
         if m.q_rank:
             cq = torch.empty((T, m.q_rank_p), **bf)
-            K.latent_rows(proj, pos, slot, cos_t, sin_t, m.rot_dim, m.rot_p, eps, q_latent=(0, m.q_rank, p[f"l{i}.q_norm"], cq), kv=kv)
-            src, kv = self._lin(cq, p[f"l{i}.w_uq"], decode, ws=1), None
+            K.latent_rows(proj, pos, slot, cos_t, sin_t, m.rot_dim, m.rot_p, eps, q_latent=(0, m.q_rank, p[f"l{i}.q_norm"], cq), kv=kv, ff=ff)
+            src, kv, ff = self._lin(cq, p[f"l{i}.w_uq"], decode, ws=1), None, None
         if isinstance(src, K.Partials):
             q = None
             nope = torch.empty((T, m.heads * m.dim_p), **bf)
@@ -386,7 +395,7 @@ class ZafopelModel(ServedDecoder):
             nope = None
         wide = None if form else torch.empty((T, m.heads, m.row_width), **bf)
         rotated = q[:, :, m.dim_p:] if form else wide[:, :, m.rank_p:]
-        K.latent_rows(src, pos, slot, cos_t, sin_t, m.rot_dim, m.rot_p, eps, kv=kv, queries=(0, m.heads, m.dim_p, nope, rotated))
+        K.latent_rows(src, pos, slot, cos_t, sin_t, m.rot_dim, m.rot_p, eps, kv=kv, queries=(0, m.heads, m.dim_p, nope, rotated), ff=ff)
         uk, uv = self._kv_maps(i)
         if form:
             return form(i, m, q)
@@ -395,14 +404,16 @@ class ZafopelModel(ServedDecoder):
         out = torch.empty((T, m.heads, m.vdim_p), **bf)
         return K.head_gemm(avg, uv, out).view(T, -1)
 
-    def _feed_forward(self, i: int, h: torch.Tensor, logits, counts: torch.Tensor, decode: bool):
-        """What the feed-forward adds to the stream, as a source of ``stream_update``."""
+    def _feed_forward(self, i: int, h: torch.Tensor, first, counts: torch.Tensor, decode: bool):
+        """What the feed-forward adds to the stream, as a source of ``stream_update``. ``first``: a mixture's router logits, or a dense one's
+        activation (None: not computed yet)."""
         p, e = self.p, self.cfg.layers[i].mlp
         if e is None:
             return None
         if isinstance(e, DenseFF):
-            return self._lin(K.ff_first(h, p[f"l{i}.w_up"], "relu2"), p[f"l{i}.w_down"], decode, ws=1)
-        ids, wts, ticket = K.moe_route(logits, e.experts, e.top, counts, sigmoid=True)
+            act = K.ff_first(h, self._ff_rows(i), "relu2") if first is None else first
+            return self._lin(act, p[f"l{i}.w_down"], decode, ws=1)
+        ids, wts, ticket = K.moe_route(first, e.experts, e.top, counts, sigmoid=True)
         r = K.moe_dispatch(h, ids, wts, ticket, counts, e.experts, weigh_inputs=True)
         act = K.moe_gemm(r.x_sorted, p[f"l{i}.w_gate_up"], r, e.experts, 0, act="swiglu")
         return K.MoEOutput(K.moe_gemm(act, p[f"l{i}.w_down"], r, e.experts, 0), r.row_of, r.weights, 0)
@@ -423,18 +434,21 @@ class ZafopelModel(ServedDecoder):
         for i, layer in enumerate(cfg.layers):
             m, e = layer.mixer, layer.mlp
             w_in, n_attn = p[f"l{i}.w_in"], m.q_in + m.kv_in
-            logits = None
-            if decode or self.f32:                                  # fp32 results: the router rides along
+            first, ff_act = None, None
+            if decode or self.f32:                                  # fp32 results: the feed-forward's rows ride along
                 proj = self._lin(h, w_in, decode)
-                if layer.router_in:
-                    logits = proj[:, n_attn:] if self.f32 else proj.columns(n_attn)
+                if isinstance(e, DenseFF):
+                    first = torch.empty((T, e.ff_p), dtype=self.dtype, device=self.device)
+                    ff_act = (n_attn, first)
+                elif e is not None:
+                    first = proj[:, n_attn:] if self.f32 else proj.columns(n_attn)
             else:
                 proj = self._lin(h, w_in[:n_attn], False)
-                if layer.router_in:
-                    logits = self._lin(h, w_in[n_attn:], False, f32_out=True)
+                if isinstance(e, InputScaledMixture):
+                    first = self._lin(h, w_in[n_attn:], False, f32_out=True)
             own = i if m.kv_from is None else m.kv_from
-            o = self._attention(i, h, proj, pos, slot, page_table, kcache[own], decode, form(i, m) if form else None, attend)
-            ff = self._feed_forward(i, h, logits, counts[i], decode)
+            o = self._attention(i, h, proj, pos, slot, page_table, kcache[own], decode, form(i, m) if form else None, attend, ff_act)
+            ff = self._feed_forward(i, h, first, counts[i], decode)
             o = self._lin(o, p[f"l{i}.wo"], decode)
             h = update(o, ff, i + 1)
             if trace is not None:
@@ -462,7 +476,7 @@ class ZafopelModel(ServedDecoder):
     def _score_latents(self, i: int, m: LatentMixer, q, kcache, page_table, slot, pos, lens, nsplit: int, scratch) -> torch.Tensor:
         cache = kcache[i if m.kv_from is None else m.kv_from]
         kw = dict(window=m.window, scale=m.scale, lens=lens, sink=self.sink[i])
-        if not self.f32 and K.latent_decode_fits(m.rank_p, m.row_width):
+        if not self.f32 and m.scale > 0 and K.latent_decode_fits(m.rank_p, m.row_width):
             return K.latent_decode(q, cache, m.rank_p, page_table, slot, pos, nsplit=nsplit, scratch=scratch, **kw)
         return K.latent_attn_rows(q, cache, m.rank_p, page_table, slot, pos, **kw)
 

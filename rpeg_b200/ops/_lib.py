@@ -95,7 +95,7 @@ _SIGNATURES = {
     "rpeg_gemm_f32": [P, P, P, I, I, I, I, I, I, P],
     "rpeg_gemm_f32_batched": [P, P, P, I, I, I, I, I, I, LL, LL, LL, I, I, P],
     "rpeg_stream_update": [I, P, I, LL, I, P, I, P, I, LL, I, P, P, I, I, LL, P, P, P, P, P, I, I, I, P],
-    "rpeg_latent_rows": [P, I, LL, I, I, P, P, P, P, I, I, F, I, I, I, P, P, I, I, I, P, P, P, I, I, I, I, P, I, P, I, I, I, P],
+    "rpeg_latent_rows": [P, I, LL, I, I, P, P, P, P, I, I, F, I, I, I, P, P, I, I, I, P, P, P, I, I, I, I, P, I, P, I, I, I, I, P, I, P],
     "rpeg_latent_gather": [P, I, P, I, P, P, P, P, I, I, P, P],
     "rpeg_latent_attn_rows": [P, P, P, I, P, P, P, P, P, I, I, I, I, I, F, I, P],
     "rpeg_latent_decode_ctas": [I, I],

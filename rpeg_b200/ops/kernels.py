@@ -928,16 +928,17 @@ def head_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, transposed
     return out
 
 
-def latent_rows(src, pos, slot, cos_t, sin_t, rot: int, rot_p: int, eps: float, *, q_latent=None, kv=None, queries=None) -> None:
+def latent_rows(src, pos, slot, cos_t, sin_t, rot: int, rot_p: int, eps: float, *, q_latent=None, kv=None, queries=None, ff=None) -> None:
     """Between a projection and latent attention, any of (column numbers refer to ``src``, an activation or ``Partials``):
       q_latent  (column, true width, weight, out [T, width_p]): weighted RMS norm of a query latent
       kv        (column, true rank, weight, cache [pages, 1, PAGE, rank_p + rot_p], page_table): the normed latent and the rotated shared key
                 part of every token into its cache row
       queries   (column, heads, dim_p, out or None, rotated [T, H, rot_p]): heads of ``[dim_p | rot_p]`` columns; the rotated parts go to the
-                (strided) view ``rotated``, which may be their place in ``src``; the others to ``out [T, H * dim_p]``, if given."""
+                (strided) view ``rotated``, which may be their place in ``src``; the others to ``out [T, H * dim_p]``, if given
+      ff        (column, out [T, ff_p]): the squared relu of ``ff_p`` columns, a feed-forward's activation."""
     part = isinstance(src, Partials)
     rows, ld = (src.M, src.N) if part else (src.shape[0], src.stride(0))
-    ref = next(t for t in (q_latent and q_latent[3], kv and kv[3], queries and queries[4]) if t is not None)
+    ref = next(t for t in (q_latent and q_latent[3], kv and kv[3], queries and queries[4], ff and ff[1]) if t is not None)
     f32 = ref.dtype == torch.float32
     if (part and f32) or (not part and src.dtype != ref.dtype):
         raise TypeError("latent_rows: source and outputs must share a dtype (split-K partials belong to the bf16 path)")
@@ -965,8 +966,14 @@ def latent_rows(src, pos, slot, cos_t, sin_t, rot: int, rot_p: int, eps: float, 
         if rot and _chk.active():
             _chk.rope("rpeg_latent_rows", pos, rows, cos_t)
         qs = (c0, H, dim_p, _ptr(out), H * dim_p, rotated.data_ptr(), rotated.stride(0), rotated.stride(1))
+    act = (0, 0, None)
+    if ff is not None:
+        c0, out = ff
+        if out.shape[0] != rows or not out.is_contiguous() or out.dtype != ref.dtype:
+            raise ValueError("latent_rows: the feed-forward's buffer does not fit")
+        act = (c0, out.shape[1], out.data_ptr())
     check(lib().rpeg_latent_rows((src.buf if part else src).data_ptr(), src.splits if part else 0, src.stride if part else 0, ld, rows, pos.data_ptr(),
-                                 slot.data_ptr(), _ptr(cos_t), _ptr(sin_t), rot, rot_p, eps, *nq, *lat, *qs, int(f32), _stream()), "rpeg_latent_rows")
+                                 slot.data_ptr(), _ptr(cos_t), _ptr(sin_t), rot, rot_p, eps, *nq, *lat, *qs, *act, int(f32), _stream()), "rpeg_latent_rows")
 
 
 def latent_gather(cache: torch.Tensor, page_table, slot, cu, off, lo, rows: int) -> torch.Tensor:
@@ -1015,7 +1022,7 @@ def latent_decode_scratch(rows: int, n_heads: int, rank_p: int, nsplit: int) -> 
 
 def latent_decode(q: torch.Tensor, cache: torch.Tensor, rank_p: int, page_table, slot, pos, *, window: int = 0, scale: float, lens=None,
                   sink: torch.Tensor | None = None, nsplit: int = 1, scratch: torch.Tensor | None = None) -> torch.Tensor:
-    """``latent_attn_rows`` on the tensor cores (bf16; sizes as ``latent_decode_fits``). The cache must hold finite numbers everywhere.
+    """``latent_attn_rows`` on the tensor cores (bf16, ``scale > 0``; sizes as ``latent_decode_fits``). The cache must hold finite numbers everywhere.
     ``nsplit > 1``: every row's pages are shared by that many CTAs (``scratch`` as ``latent_decode_scratch``)."""
     _req(q, torch.bfloat16, "q")
     _req(cache, torch.bfloat16, "cache")

@@ -395,7 +395,7 @@ def test_mixture_with_scaled_inputs(cuda_device, dtype, T, E, top, ff, width):
     scores, chosen = O.route(h.double(), td, "l0.mlp.", cfg["layers"][0]["mlp"]["router"])
     hd = _pad(h.to(dtype), m.cfg.width_p).to(cuda_device)
     mx = m.cfg.layers[0].mixer
-    router = m.p["l0.w_in"][mx.q_in + mx.kv_in:]
+    router = m._ff_rows(0)
     logits = [m._lin(hd, router, False, f32_out=True)]
     if T <= 256 and dtype == torch.bfloat16:                 # decode: the router's columns of the stacked projection's partials
         logits.append(m._lin(hd, m.p["l0.w_in"], True).columns(mx.q_in + mx.kv_in))
@@ -424,8 +424,15 @@ def test_dense_feed_forward(cuda_device, dtype, T, ff, width):
     h = torch.randn(T, width, generator=torch.Generator().manual_seed(3)).bfloat16()
     want = O.dense(h.double(), {n: v.double() for n, v in t.items()}, "l0.mlp.")
     hd = _pad(h.to(dtype), m.cfg.width_p).to(cuda_device)
+    mx, fp = m.cfg.layers[0].mixer, _p8(ff)
     for decode in ((False, True) if dtype == torch.bfloat16 and T <= 256 else (False,)):
-        out = m._feed_forward(0, hd, None, None, decode)
+        first = None
+        if decode or dtype == torch.float32:                 # the first product comes with the layer's projection
+            first = torch.full((T, fp), 5.0, dtype=dtype, device=cuda_device)
+            K.latent_rows(m._lin(hd, m.p["l0.w_in"], decode), torch.zeros(T, dtype=torch.int32, device=cuda_device), torch.zeros(T, dtype=torch.int32, device=cuda_device),
+                          None, None, 0, 8, 1e-5, ff=(mx.q_in + mx.kv_in, first))
+            assert D.worst_row(first[:, :ff], torch.relu(h.double() @ t["l0.mlp.up"].double().T) ** 2) < TOL[dtype] and first[:, ff:].abs().sum() == 0
+        out = m._feed_forward(0, hd, first, None, decode)
         out = out.reduce() if isinstance(out, K.Partials) else out
         assert D.worst_row(out[:, :width], want) < TOL[dtype] and out[:, width:].abs().sum() == 0
 

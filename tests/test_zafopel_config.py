@@ -78,7 +78,7 @@ def test_weights_land_in_padded_layout(tmp_path):
     assert p["l2.w_in"].shape == (7 * 48 + 8, 104) and "l2.kv_norm" not in p and p["l3.w_in"].shape == (24, 104)
     gu = p["l0.w_gate_up"]
     assert gu.shape == (6, 80, 104) and torch.equal(gu[4, :36, :w], t["l0.mlp.e4.gate"]) and torch.equal(gu[4, 40:76, :w], t["l0.mlp.e4.up"])
-    assert torch.equal(p["l0.w_down"][4, :w, :36], t["l0.mlp.e4.down"]) and torch.equal(p["l1.w_up"][:50, :w], t["l1.mlp.up"])
+    assert torch.equal(p["l0.w_down"][4, :w, :36], t["l0.mlp.e4.down"]) and torch.equal(m._ff_rows(1)[:50, :w], t["l1.mlp.up"])
     assert torch.equal(m.alpha.bfloat16(), torch.stack([t[f"l{i}.norm1.alpha"] for i in range(5)] + [t["final.norm.alpha"]]))
     assert torch.equal(p["l2.norm1.b"][:w], t["l2.norm1.b"]) and torch.equal(m.sink[3], t["l3.mix.sink"].float()) and m.sink[1] is None
     assert torch.equal(p["head"][:301, :w], t["head"]) and torch.equal(p["embed"][:301, :w], t["embed"])
