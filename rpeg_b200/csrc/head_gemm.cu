@@ -65,25 +65,26 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
           tma_load_3d(sb, &tmap_b, &full_bar[st], kb * HG_BK, n0, h);
         }
       };
-      const int pre = stages;
-      for (int kb = 0; kb < pre; ++kb) load_b(kb, kb);         // weights do not depend on the kernel before
+      for (int kb = 0; kb < stages; ++kb) load_b(kb, kb);      // weights do not depend on the kernel before
       griddep_wait();
-      for (int kb = 0; kb < num_kb; ++kb) {
-        const int st = kb % stages;
-        if (kb >= pre) {
-          if (!mbar_wait(&empty_bar[st], (static_cast<uint32_t>(kb / stages) & 1u) ^ 1u, abort_flag, status, 1000)) break;
-          load_b(kb, st);
-        }
+      for (int kb = 0; kb < stages; ++kb) tma_load_3d(smem + kb * Cfg::STAGE_BYTES, &tmap_a, &full_bar[kb], kb * HG_BK, h, m0);
+      int st = 0;
+      uint32_t phase = 0u;
+      for (int kb = stages; kb < num_kb; ++kb) {
+        if (!mbar_wait(&empty_bar[st], phase, abort_flag, status, 1000)) break;
+        load_b(kb, st);
         tma_load_3d(smem + st * Cfg::STAGE_BYTES, &tmap_a, &full_bar[st], kb * HG_BK, h, m0);
+        if (++st == stages) { st = 0; phase ^= 1u; }
       }
     }
   } else if (warp == 1) {
     const bool leader = elect_one();               // all lanes run the loop, one issues
     constexpr uint32_t idesc = make_idesc_bf16(HG_BM, BN, 0, B_KN ? 1 : 0);
     bool ok = true;
+    int st = 0;
+    uint32_t phase = 0u;
     for (int kb = 0; kb < num_kb; ++kb) {
-      const int st = kb % stages;
-      if (!__all_sync(0xffffffffu, mbar_wait(&full_bar[st], static_cast<uint32_t>(kb / stages) & 1u, abort_flag, status, 1010))) { ok = false; break; }
+      if (!__all_sync(0xffffffffu, mbar_wait(&full_bar[st], phase, abort_flag, status, 1010))) { ok = false; break; }
       tc_fence_after_sync();
       const uint32_t sa = smem_u32(smem + st * Cfg::STAGE_BYTES), sb = sa + Cfg::A_BYTES;
 #pragma unroll
@@ -93,6 +94,7 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                        B_KN ? make_smem_desc_sw128(sb + k * 2048, 64 * HG_BK * 2, 1024) : make_smem_desc_sw128(sb + k * 32, 16, 1024), idesc,
                        (kb | k) != 0 ? 1u : 0u);
       if (leader) umma_commit(&empty_bar[st]);
+      if (++st == stages) { st = 0; phase ^= 1u; }
     }
     if (ok && leader) umma_commit(done_bar);
   } else {

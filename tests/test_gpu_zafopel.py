@@ -107,7 +107,7 @@ def test_tanh_is_accurate_over_its_range(cuda_device):
 # --------------------------------------------------------------------------- latents, rotations, per-head products
 @pytest.mark.parametrize("dtype", DT)
 @pytest.mark.parametrize("partials", [False, True])
-@pytest.mark.parametrize("H,dim,rot,rank,nq", [(5, 20, 12, 36, 44), (3, 64, 32, 96, 0), (1, 8, 2, 200, 1500), (4, 40, 0, 24, 8)])
+@pytest.mark.parametrize("H,dim,rot,rank,nq", [(5, 20, 12, 36, 44), (3, 48, 32, 88, 0), (1, 8, 2, 200, 1500), (4, 40, 0, 24, 8)])
 def test_latent_rows(cuda_device, dtype, partials, H, dim, rot, rank, nq):
     if partials and dtype == torch.float32:
         pytest.skip("split-K partials belong to the bf16 path")
@@ -206,7 +206,7 @@ def _score(kernel, q, cache, rank, table, slot, pos, window, scale, sink, lens=N
 
 
 @pytest.mark.parametrize("kernel", ["rows f32", "rows bf16", "tensor", "tensor split"])
-@pytest.mark.parametrize("H,rank,W,window,sink", [(6, 96, 128, 0, True), (5, 40, 56, 37, False), (33, 512, 576, 0, True), (32, 512, 576, 64, False), (70, 136, 144, 65, True),
+@pytest.mark.parametrize("H,rank,W,window,sink", [(7, 88, 112, 0, True), (5, 40, 56, 37, False), (33, 512, 576, 0, True), (32, 512, 576, 64, False), (70, 136, 144, 65, True),
                                                   (1, 8, 8, 1, False), (16, 320, 384, 200, True), (3, 256, 288, 2, True), (9, 64, 576, 300, False)])
 def test_scores_on_cached_rows(cuda_device, kernel, H, rank, W, window, sink):
     """Query rows that stand anywhere, of two requests of unequal length, every row against the oracle."""
@@ -284,7 +284,7 @@ def _prefill(cuda_device, lens, starts, H, dim, rot, vdim, window, scale, sink, 
     return out.view(T, H, vp)[..., :vdim].reshape(T, -1), torch.cat(wants)
 
 
-@pytest.mark.parametrize("H,dim,rot,vdim,window,sink", [(6, 64, 32, 64, 0, True), (2, 20, 12, 28, 37, False), (3, 128, 64, 128, 0, True), (1, 128, 64, 96, 200, True), (2, 40, 2, 72, 1, False),
+@pytest.mark.parametrize("H,dim,rot,vdim,window,sink", [(5, 56, 24, 56, 0, True), (2, 20, 12, 28, 37, False), (3, 128, 64, 128, 0, True), (1, 128, 64, 96, 200, True), (2, 40, 2, 72, 1, False),
                                                         (2, 72, 16, 16, 64, True), (1, 192, 0, 128, 129, False), (2, 64, 128, 64, 5, True), (4, 8, 8, 8, 300, False)])
 def test_prompt_attention_on_formed_keys(cuda_device, H, dim, rot, vdim, window, sink):
     g = torch.Generator().manual_seed(dim + window)
@@ -381,7 +381,7 @@ def test_latent_gather(cuda_device, dtype):
 
 # --------------------------------------------------------------------------- feed-forwards
 @pytest.mark.parametrize("dtype", DT)
-@pytest.mark.parametrize("T,E,top,ff,width", [(1, 6, 3, 36, 100), (37, 8, 1, 96, 64), (300, 5, 5, 40, 72), (200, 64, 6, 32, 128), (260, 1, 1, 200, 264), (90, 300, 4, 16, 48)])
+@pytest.mark.parametrize("T,E,top,ff,width", [(1, 6, 3, 36, 100), (37, 7, 1, 88, 64), (300, 5, 5, 40, 72), (200, 64, 6, 32, 128), (260, 1, 1, 200, 264), (90, 300, 4, 16, 48)])
 def test_mixture_with_scaled_inputs(cuda_device, dtype, T, E, top, ff, width):
     cfg = C.config(width, 32, [C.layer(1, 8, 2, 8, 8, 1.0, 100.0, window=4, mlp=C.moe(E, top, ff))])
     t = C.tensors(cfg, T + E)
@@ -415,7 +415,7 @@ def test_mixture_with_scaled_inputs(cuda_device, dtype, T, E, top, ff, width):
 
 
 @pytest.mark.parametrize("dtype", DT)
-@pytest.mark.parametrize("T,ff,width", [(1, 50, 100), (130, 256, 64), (40, 1000, 136), (300, 24, 1030)])
+@pytest.mark.parametrize("T,ff,width", [(1, 50, 100), (130, 264, 64), (40, 1000, 136), (300, 24, 1030)])
 def test_dense_feed_forward(cuda_device, dtype, T, ff, width):
     cfg = C.config(width, 32, [C.layer(1, 8, 2, 8, 8, 1.0, 100.0, window=4, mlp=C.dense(ff))])
     t = C.tensors(cfg, ff)

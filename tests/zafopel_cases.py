@@ -46,7 +46,7 @@ def sliding():
     """Windows everywhere (no multiples of a page), so old pages go back while a request runs."""
     return config(128, 256, [
         layer(8, 64, 32, 64, 128, 0.12, 10000.0, window=90, mlp=moe(8, 2, 64)),
-        layer(4, 48, 32, 40, 128, 0.15, 10000.0, window=70, kv_from=0, mlp=dense(256)),
+        layer(4, 48, 32, 40, 128, 0.15, 10000.0, window=70, kv_from=0, mlp=dense(248)),
         layer(8, 64, 32, 64, 128, 0.12, 10000.0, window=90, mlp=moe(8, 2, 64)),
     ], 1e-6)
 
